@@ -1,4 +1,5 @@
-"""ctypes binding of libvuib200 (include/vuib200.h) and its in-tree build.
+"""ctypes bindings of libvuib200 (include/vuib200.h) and libvuib200_lm (include/vuib200_lm.h), and their
+in-tree build.  Each library is compiled and loaded on its own: a token model needs only the second.
 
 There is no fallback: if the shared library is missing and cannot be built, or a
 call returns a non-zero status, this module raises.
@@ -14,17 +15,24 @@ import subprocess
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _ROOT = os.path.dirname(_HERE)
 LIB_PATH = os.path.join(_HERE, "libvuib200.so")
+LM_LIB_PATH = os.path.join(_HERE, "libvuib200_lm.so")
 _CSRC = os.path.join(_HERE, "csrc")
 _OBJ = os.path.join(_CSRC, "_obj")
 _API_H = os.path.join(_ROOT, "include", "vuib200.h")
+_LM_API_H = os.path.join(_ROOT, "include", "vuib200_lm.h")
 # translation unit -> the headers it includes (a unit is recompiled when one of them changes)
+_COMMON = ["decode_kernels.cuh", "tc_gemm.cuh", "host_common.cuh"]
 UNITS = {
-    "vuib200.cu": ["decode_kernels.cuh", "tc_gemm.cuh", "fused_blocks.cuh", "depth_group.cuh", "prefill_attn.cuh"],
+    "vuib200.cu": [*_COMMON, "fused_blocks.cuh", "depth_group.cuh", "prefill_attn.cuh"],
     "codec.cu": ["codec_kernels.cuh"],
     "codec_enc.cu": ["codec_enc_kernels.cuh"],
+    "lm.cu": [*_COMMON, "lm_kernels.cuh", "latent_attn.cuh", "latent_prefill.cuh"],
 }
-SOURCES = [os.path.join(_CSRC, u) for u in UNITS]
-HEADERS = sorted({os.path.join(_CSRC, h) for hs in UNITS.values() for h in hs}) + [_API_H]
+# library -> (its units, the API headers they include)
+LIBRARIES = {
+    LIB_PATH: (["vuib200.cu", "codec.cu", "codec_enc.cu"], [_API_H]),
+    LM_LIB_PATH: (["lm.cu"], [_API_H, _LM_API_H]),
+}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC",
@@ -201,42 +209,93 @@ SYMBOLS = {
     "vuib_codec_enc_launch_count": (C.c_int64, [_P]),
 }
 
+# ---------------------------------------------------------------------------- include/vuib200_lm.h
+LM_BF16, LM_F32 = 0, 1
+LM_MIX_LATENT = 1
+LM_MLP_NONE, LM_MLP_CLAMPED_GLU = 0, 1
 
-def _src_hash() -> str:
+
+class VuibLmConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "n_layers", "dtype", "n_slots", "max_seq", "max_rows",
+                                         "max_prefill_rows")] + [("norm_eps", C.c_float), ("embed_scale", C.c_float)]
+
+
+class VuibLmLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "mlp", "heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank", "q_rank",
+                                         "ff")] + [(n, C.c_float) for n in ("scale", "mlp_limit", "mlp_slope", "mlp_shift")]
+
+
+class VuibLmDims(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("k_in", "n_dq", "n_kv", "n_gate", "n_mlp", "n_in", "rp", "rotp", "dp", "k_q", "n_q",
+                                         "k_out", "off_y", "n_out", "x_ok", "dimp", "vdp", "n_xq", "k_kv", "n_xkv")]
+
+
+class VuibLmLayerWeights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("norm1_w", "norm1_b", "norm2_w", "norm2_b", "q_norm", "kv_norm", "w_in", "w_q",
+                                          "w_uv", "w_out", "w_xq", "w_xkv", "trig")]
+
+
+class VuibLmHeadWeights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("embed", "final_w", "final_b", "head")]
+
+
+LM_SYMBOLS = {
+    "vuib_lm_abi_version": (C.c_int32, []),
+    "vuib_lm_create": (C.c_int32, [C.POINTER(VuibLmConfig), C.POINTER(VuibLmLayer), C.POINTER(_P)]),
+    "vuib_lm_destroy": (C.c_int32, [_P]),
+    "vuib_lm_last_error": (C.c_int32, [_P, C.c_char_p, C.c_size_t]),
+    "vuib_lm_layer_dims": (C.c_int32, [_P, C.c_int32, C.POINTER(VuibLmDims)]),
+    "vuib_lm_workspace_bytes": (C.c_int32, [_P, C.POINTER(C.c_size_t)]),
+    "vuib_lm_bind_workspace": (C.c_int32, [_P, _P, C.c_size_t]),
+    "vuib_lm_bind_weights": (C.c_int32, [_P, C.POINTER(VuibLmHeadWeights), C.POINTER(VuibLmLayerWeights)]),
+    "vuib_lm_bind_cache": (C.c_int32, [_P, C.POINTER(_P), _P]),
+    "vuib_lm_prefill": (C.c_int32, [_P, C.c_int32, C.POINTER(C.c_int32), C.POINTER(C.c_int32), C.POINTER(C.c_int32), _P,
+                                    C.c_int32, _P, _P, _P]),
+    "vuib_lm_decode": (C.c_int32, [_P, C.c_int32, _P, _P, _P, _P, _P]),
+    "vuib_lm_set_sampling": (C.c_int32, [_P, C.POINTER(VuibSampling), _P]),
+    "vuib_lm_sample": (C.c_int32, [_P, C.c_int32, _P, _P, _P, _P]),
+    "vuib_lm_reset_slot": (C.c_int32, [_P, C.c_int32, _P]),
+    "vuib_lm_set_taps": (C.c_int32, [_P, _P]),
+    "vuib_lm_set_expand_min": (C.c_int32, [_P, C.c_int32]),
+    "vuib_lm_set_wait_limit": (C.c_int32, [_P, C.c_uint32]),
+    "vuib_lm_check_device_flag": (C.c_int32, [_P, _P]),
+    "vuib_lm_launch_count": (C.c_int64, [_P]),
+}
+
+
+def _hash_files(paths) -> str:
     import hashlib
 
     h = hashlib.sha256()
-    for p in SOURCES + HEADERS:
+    for p in paths:
         with open(p, "rb") as f:
             h.update(f.read())
     h.update(" ".join(NVCC_FLAGS).encode())
     return h.hexdigest()
 
 
-def _stale() -> bool:
+def _unit_files(unit: str, api) -> list[str]:
+    return [os.path.join(_CSRC, unit)] + [os.path.join(_CSRC, x) for x in UNITS[unit]] + list(api)
+
+
+def _src_hash(path: str) -> str:
+    units, api = LIBRARIES[path]
+    return _hash_files(sorted({f for u in units for f in _unit_files(u, api)}))
+
+
+def _stale(path: str) -> bool:
     """True when the .so is missing or was built from other sources (a content
     hash beside the .so decides, not mtimes, which a copy of the tree changes)."""
-    if not os.path.exists(LIB_PATH) or not os.path.exists(LIB_PATH + ".srchash"):
+    if not os.path.exists(path) or not os.path.exists(path + ".srchash"):
         return True
-    with open(LIB_PATH + ".srchash") as f:
-        return f.read().strip() != _src_hash()
+    with open(path + ".srchash") as f:
+        return f.read().strip() != _src_hash(path)
 
 
-def _unit_hash(unit: str) -> str:
-    import hashlib
-
-    h = hashlib.sha256()
-    for p in [os.path.join(_CSRC, unit)] + [os.path.join(_CSRC, x) for x in UNITS[unit]] + [_API_H]:
-        with open(p, "rb") as f:
-            h.update(f.read())
-    h.update(" ".join(NVCC_FLAGS).encode())
-    return h.hexdigest()
-
-
-def _compile_unit(nvcc: str, unit: str, verbose: bool) -> str:
+def _compile_unit(nvcc: str, unit: str, api, verbose: bool) -> str:
     """Compile one translation unit to an object file, unless an object of the same inputs exists."""
     obj = os.path.join(_OBJ, unit + ".o")
-    stamp, want = obj + ".srchash", _unit_hash(unit)
+    stamp, want = obj + ".srchash", _hash_files(_unit_files(unit, api))
     if os.path.exists(obj) and os.path.exists(stamp):
         with open(stamp) as f:
             if f.read().strip() == want:
@@ -254,55 +313,67 @@ def _compile_unit(nvcc: str, unit: str, verbose: bool) -> str:
     return obj
 
 
-def build_library(force: bool = False, verbose: bool = False) -> str:
-    """Compile csrc/*.cu for sm_100a into vui_b200/libvuib200.so (in-tree): one object per
-    translation unit, compiled side by side, then one link."""
-    if not force and not _stale():
-        return LIB_PATH
+def build_library(force: bool = False, verbose: bool = False, paths=None) -> str:
+    """Compile csrc/*.cu for sm_100a into the in-tree libraries (`paths`: all by default): one object per
+    translation unit, compiled side by side, then one link per library.  Returns the first path."""
+    paths = list(LIBRARIES) if paths is None else list(paths)
+    todo = [p for p in paths if force or _stale(p)]
+    if not todo:
+        return paths[0]
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(nvcc):
-        raise RuntimeError("libvuib200.so is missing or stale and nvcc was not found to build it")
+        raise RuntimeError(f"{os.path.basename(todo[0])} is missing or stale and nvcc was not found to build it")
     os.makedirs(_OBJ, exist_ok=True)
+    units = [(u, LIBRARIES[p][1]) for p in todo for u in LIBRARIES[p][0]]
     if force:
-        for u in UNITS:
+        for u, _ in units:
             if os.path.exists(os.path.join(_OBJ, u + ".o.srchash")):
                 os.remove(os.path.join(_OBJ, u + ".o.srchash"))
     from concurrent.futures import ThreadPoolExecutor
 
-    with ThreadPoolExecutor(max_workers=len(UNITS)) as pool:
-        objs = list(pool.map(lambda u: _compile_unit(nvcc, u, verbose), UNITS))
-    res = subprocess.run([nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-shared",
-                          "-o", LIB_PATH, *objs], capture_output=True, text=True)
-    if res.returncode != 0:
-        raise RuntimeError(f"nvcc link failed:\n{res.stdout}\n{res.stderr}")
-    with open(LIB_PATH + ".srchash", "w") as f:
-        f.write(_src_hash())
-    return LIB_PATH
+    with ThreadPoolExecutor(max_workers=len(units)) as pool:
+        objs = dict(zip([u for u, _ in units], pool.map(lambda a: _compile_unit(nvcc, a[0], a[1], verbose), units)))
+    for p in todo:
+        part = f"{p}.{os.getpid()}.part"
+        res = subprocess.run([nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-shared",
+                              "-o", part, *[objs[u] for u in LIBRARIES[p][0]]], capture_output=True, text=True)
+        if res.returncode != 0:
+            raise RuntimeError(f"nvcc link failed:\n{res.stdout}\n{res.stderr}")
+        os.replace(part, p)
+        with open(p + ".srchash", "w") as f:
+            f.write(_src_hash(p))
+    return paths[0]
 
 
-_lib = None
+_loaded: dict[str, C.CDLL] = {}
 
 
-def load() -> C.CDLL:
-    """Load the library (building it when the sources are newer) and type every symbol."""
-    global _lib
-    if _lib is not None:
-        return _lib
-    if _stale() and (shutil.which("nvcc") or os.path.exists("/usr/local/cuda/bin/nvcc")):
-        build_library()
-    if not os.path.exists(LIB_PATH):
-        raise RuntimeError(
-            f"{LIB_PATH} not found: build it with `python -c 'import __graft_entry__ as g; g.build()'`"
-        )
-    lib = C.CDLL(LIB_PATH)
-    for name, (res, args) in SYMBOLS.items():
+def _load(path: str, symbols: dict, version: str) -> C.CDLL:
+    if path in _loaded:
+        return _loaded[path]
+    if _stale(path) and (shutil.which("nvcc") or os.path.exists("/usr/local/cuda/bin/nvcc")):
+        build_library(paths=[path])
+    if not os.path.exists(path):
+        raise RuntimeError(f"{path} not found: build it with `python -c 'import __graft_entry__ as g; g.build()'`")
+    lib = C.CDLL(path)
+    for name, (res, args) in symbols.items():
         fn = getattr(lib, name)  # AttributeError if the export is missing
         fn.restype = res
         fn.argtypes = args
-    if lib.vuib_abi_version() != 1:
-        raise RuntimeError("libvuib200 ABI version mismatch")
-    _lib = lib
+    if getattr(lib, version)() != 1:
+        raise RuntimeError(f"{os.path.basename(path)}: ABI version mismatch")
+    _loaded[path] = lib
     return lib
+
+
+def load() -> C.CDLL:
+    """Load libvuib200 (building it when the sources are newer) and type every symbol."""
+    return _load(LIB_PATH, SYMBOLS, "vuib_abi_version")
+
+
+def load_lm() -> C.CDLL:
+    """The same for libvuib200_lm."""
+    return _load(LM_LIB_PATH, LM_SYMBOLS, "vuib_lm_abi_version")
 
 
 class VuibError(RuntimeError):
@@ -311,10 +382,11 @@ class VuibError(RuntimeError):
         self.code = code
 
 
-def check(handle, code: int) -> None:
+def check(handle, code: int, last_error=None) -> None:
+    """Raise for a non-zero status; `last_error` is the handle's own text function (libvuib200's by default)."""
     if code == 0:
         return
     buf = C.create_string_buffer(256)
     if handle:
-        load().vuib_last_error(handle, buf, 256)
+        (last_error or load().vuib_last_error)(handle, buf, 256)
     raise VuibError(code, buf.value.decode() or "(no message)")

@@ -306,6 +306,7 @@ struct TcArgs {
     int32_t* flag;
     unsigned long long* dbg;  // optional: device-clock stamps of CTA (0,0) (profiling aid)
     unsigned spin_limit;      // polls after which a wait gives up and records FLAG_TC_TIMEOUT
+    int x_split_tile, x_split_row;  // weight tiles >= x_split_tile multiply the rows x_split_row further down in X
 };
 
 __device__ __forceinline__ void tc_stamp(const TcArgs& a, int i) {
@@ -333,6 +334,7 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapA0, const __grid_constant__ CUt
     const int tile_id = blockIdx.z * a.tiles + tile;  // index of the (block, tile) pair in the split-K scratch
     const int all_tiles = gridDim.z * a.tiles;
     const Epi ep = ep_all.shifted(m_base);
+    const int x_row = m_base + (tile >= a.x_split_tile ? a.x_split_row : 0);  // first row of X this CTA multiplies
     tc_stamp(a, 0);
     const int stages = a.stages;  // <= smallest chunk count of any split
     const uint32_t a_bytes = TC_TILE_N * TC_KCHUNK * 2, b_bytes = (uint32_t)a.Mpad * TC_KCHUNK * 2;
@@ -381,7 +383,7 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapA0, const __grid_constant__ CUt
         }
         pdl_wait();
         for (int c = 0; c < stages; ++c)
-            tma_load_2d(base + (size_t)c * stage_bytes + a_bytes, &mapX, (k_first + c) * TC_KCHUNK, m_base, &bar_full[c]);
+            tma_load_2d(base + (size_t)c * stage_bytes + a_bytes, &mapX, (k_first + c) * TC_KCHUNK, x_row, &bar_full[c]);
         for (int c = stages; c < n_chunks; ++c) {
             const int s = c % stages;
             if (!mbar_wait(&bar_empty[s], ((c / stages) & 1) ^ 1, 4 * a.spin_limit)) { s_bad = 1; break; }
@@ -389,7 +391,7 @@ k_gemm_tc(const __grid_constant__ CUtensorMap mapA0, const __grid_constant__ CUt
             mbar_expect_tx(&bar_full[s], a_bytes + b_bytes);
             tma_load_2d(st, &mapA0, (k_first + c) * TC_KCHUNK, rowA0, &bar_full[s]);
             tma_load_2d(st + a_bytes / 2, &mapA1, (k_first + c) * TC_KCHUNK, rowA1, &bar_full[s]);
-            tma_load_2d(st + a_bytes, &mapX, (k_first + c) * TC_KCHUNK, m_base, &bar_full[s]);
+            tma_load_2d(st + a_bytes, &mapX, (k_first + c) * TC_KCHUNK, x_row, &bar_full[s]);
         }
       }
       __syncwarp();

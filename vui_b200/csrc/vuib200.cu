@@ -13,6 +13,7 @@
 
 #include "decode_kernels.cuh"
 #include "tc_gemm.cuh"
+#include "host_common.cuh"
 #include "fused_blocks.cuh"
 #include "depth_group.cuh"
 #include "prefill_attn.cuh"
@@ -31,7 +32,6 @@ struct WsLayout {
     size_t total;
 };
 
-constexpr int TC_PARTIAL_TILES = 224;  // most (tile, split) pairs of one GEMM launch
 constexpr int FB_MLP_TH_BACKBONE = 512, FB_MLP_U_BACKBONE = 32;  // threads, hidden units per CTA of the MLP block
 constexpr int FB_MLP_TH_DEPTH = 256, FB_MLP_U_DEPTH = 16;
 constexpr int FUSED_MAX_PARTS = 16;     // most partial rows a fused block leaves (clusters of its grid)
@@ -118,8 +118,6 @@ static int32_t fail(VuibEngine* e, int32_t code, const char* fmt, ...) {
     return code;
 }
 
-static size_t align_up(size_t v) { return (v + 255) & ~(size_t)255; }
-
 static void make_layout(VuibEngine* e) {
     const VuibConfig& c = e->cfg;
     WsLayout& L = e->lay;
@@ -154,8 +152,8 @@ static void make_layout(VuibEngine* e) {
     L.xn = take(R * (size_t)(c.ffn > c.d_model ? c.ffn : c.d_model) * 2);
     L.rq_xn = take(2 * RB * rd * 2);
     L.rq_attn = take(2 * RB * rd * 2);
-    L.tc_partial = take((size_t)(TC_PARTIAL_TILES + 80) * TC_TILE_N * (R < 256 ? ((R + 15) / 16) * 16 : 256) * 4);
-    L.tc_counters = take(2 * 256 * 4);
+    L.tc_partial = take(tc_partial_bytes(R));
+    L.tc_counters = take(2 * TC_COUNTERS * 4);
     L.dg_layers = L.dg_head = 0;
     if (c.rq_d_model == DG_D && c.rq_n_heads == DG_CL && c.rq_n_layers <= DG_LAYERS && c.rq_ffn % DG_CL == 0 &&
         c.rq_ffn / DG_CL <= 192 && c.codebook_size == DG_CL * 256) {
@@ -176,51 +174,6 @@ static void make_layout(VuibEngine* e) {
     L.att_tiles = take(2 * R * 4);
     L.att_ntiles = take(256);
     L.total = off;
-}
-
-// Launch with the programmatic-stream-serialization attribute (see pdl_wait in
-// decode_kernels.cuh) unless VUIB_NO_PDL is set in the environment.
-static bool env_off(const char* name) {
-    const char* s = getenv(name);
-    return s && s[0] && s[0] != '0';
-}
-
-static bool pdl_enabled() {
-    static int v = -1;
-    if (v < 0) {
-        const char* s = getenv("VUIB_NO_PDL");
-        v = (s && s[0] && s[0] != '0') ? 0 : 1;
-    }
-    return v == 1;
-}
-
-// Every kernel of a frame asks for the same (largest) shared-memory carve-out.  The tensor-core
-// GEMM needs ~100-200 KB of shared memory and the small kernels between two GEMMs need almost
-// none; left to their own preferences the SMs would re-partition L1/shared memory at every
-// switch, which drains them and blocks the overlap of consecutive launches.
-static void prefer_max_smem(const void* kern) {
-    static std::mutex mu;
-    static std::unordered_set<const void*> done;
-    std::lock_guard<std::mutex> lock(mu);
-    if (done.insert(kern).second)
-        cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
-}
-
-template <class... KArgs, class... Args>
-static cudaError_t launch(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s,
-                          Args... args) {
-    prefer_max_smem(reinterpret_cast<const void*>(kern));
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = s;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = pdl_enabled() ? 1 : 0;
-    return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
 }
 
 template <class T>
@@ -423,51 +376,6 @@ extern "C" int32_t vuib_set_taps(VuibEngine* e, void* layer_hidden_dev, void* rq
 // ---------------------------------------------------------------------------
 // Tensor-core path (tc_gemm.cuh) for five rows and more: many streams, prefill.
 // ---------------------------------------------------------------------------
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                                  const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = nullptr;
-    static bool tried = false;
-    if (!tried) {
-        tried = true;
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-            q == cudaDriverEntryPointSuccess)
-            fn = reinterpret_cast<EncodeTiledFn>(p);
-    }
-    return fn;
-}
-
-// 2-D bf16 row-major (rows, cols) tensor, boxes of box_rows x 64 columns, 128-byte swizzle.
-static bool make_map(CUtensorMap* m, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows) {
-    EncodeTiledFn fn = encode_tiled_fn();
-    if (!fn) return false;
-    cuuint64_t dims[2] = {cols, rows};
-    cuuint64_t strides[1] = {cols * 2};
-    cuuint32_t box[2] = {TC_KCHUNK, box_rows};
-    cuuint32_t estr[2] = {1, 1};
-    return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
-              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
-// 2-D bf16 row-major (rows, cols) tensor, dense boxes of box_rows x box_cols, no swizzle.
-static bool make_map_plain(CUtensorMap* m, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows,
-                           uint32_t box_cols) {
-    EncodeTiledFn fn = encode_tiled_fn();
-    if (!fn || box_rows > 256 || box_cols > 256) return false;
-    cuuint64_t dims[2] = {cols, rows};
-    cuuint64_t strides[1] = {cols * 2};
-    cuuint32_t box[2] = {box_cols, box_rows};
-    cuuint32_t estr[2] = {1, 1};
-    return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
-              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 static void build_tc_maps(VuibEngine* e) {
     delete e->tc;
     e->tc = nullptr;
@@ -545,72 +453,15 @@ static bool tc_ok(VuibEngine* e, int M) {
     return M > 4 && e->tc && !env_off("VUIB_NO_TC");
 }
 
-// D = W X^T over all M rows in blocks of <= 256, epilogue ep (see tc_gemm.cuh).
-//  units: weight rows (N, multiple of 128) or, for the paired SwiGLU form, hidden units (multiple of 64).
+// The engine's scratch in front of tc_gemm_launch (host_common.cuh).
 template <class Epi>
 static int32_t tc_gemm(VuibEngine* e, const CUtensorMap& a0, const CUtensorMap& a1, const bf16* X, int M, int K,
                        int units, int row_off, const Epi& ep, cudaStream_t s) {
     const WsLayout& L = e->lay;
-    const int tiles = Epi::PAIRED ? units / 64 : units / TC_TILE_N;
-    const int chunks_total = K / TC_KCHUNK;
-    // Split K over enough CTAs to occupy the SMs (one MMA of this shape takes ~96 ns whatever the
-    // batch, so the tensor pipe of ONE SM consumes weights at only ~42 GB/s).  The CTAs of a tile
-    // meet on a counter, so the grid must be resident at once: at most two CTAs per SM.
-    if (e->num_sms == 0) {
-        int dev = 0;
-        CK(cudaGetDevice(&dev));
-        CK(cudaDeviceGetAttribute(&e->num_sms, cudaDevAttrMultiProcessorCount, dev));
-    }
-    // Row blocks: up to 256 activation rows per CTA; a prefill of more rows is ONE launch whose grid's z
-    // dimension walks the blocks (every weight tile is then read by its row blocks back to back and stays in
-    // L2), not one launch per block.
-    const int Mpad = M <= 256 ? (M + 15) / 16 * 16 : 256;
-    const int m_blocks = (M + Mpad - 1) / Mpad;
-    int splits = 1;
-    for (int d = 2; d <= 16; d *= 2) {
-        if (d > chunks_total || tiles * m_blocks * d > e->num_sms + e->num_sms / 2) break;
-        if (Epi::PAIRED && d == 2) continue;
-        splits = d;
-    }
-    const int max_smem = 202 * 1024;
-    {   // a function attribute belongs to one device's copy of the kernel: set it once per device
-        static std::mutex mu;
-        static bool attr_set[64];
-        int dev = 0;
-        CK(cudaGetDevice(&dev));
-        std::lock_guard<std::mutex> lock(mu);
-        if (dev < 0 || dev >= 64 || !attr_set[dev]) {
-            CK(cudaFuncSetAttribute(k_gemm_tc<Epi>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem));
-            if (dev >= 0 && dev < 64) attr_set[dev] = true;
-        }
-    }
-    CUtensorMap mx;
-    if (!make_map(&mx, X, M, K, Mpad)) return fail(e, VUIB_ERR_CUDA, "cuTensorMapEncodeTiled failed");
-    TcArgs ta;
-    ta.N = units;
-    ta.row_off = row_off;
-    ta.M = M;
-    ta.Mpad = Mpad;
-    ta.chunks = chunks_total;
-    ta.splits = splits;
-    ta.tiles = tiles;
-    ta.partial = wsp<float>(e, L.tc_partial);
-    ta.counters = wsp<int32_t>(e, L.tc_counters);
-    ta.flag = wsp<int32_t>(e, L.flag);
-    ta.dbg = env_off("VUIB_TRACE") ? wsp<unsigned long long>(e, L.trace) : nullptr;
-    ta.spin_limit = e->spin_limit;
-    const int min_chunks = chunks_total / splits;  // the shortest split
-    const size_t stage_bytes = TC_TILE_N * TC_KCHUNK * 2 + ((Mpad * TC_KCHUNK * 2 + 1023) & ~1023);
-    const size_t epi_bytes = Epi::STAGED ? (size_t)Mpad * TC_EPI_BYTES_PER_M : 0;
-    // two CTAs per SM when split (all CTAs of the grid must be resident), the whole SM otherwise
-    const size_t budget = (splits > 1 ? 100 : 200) * 1024;
-    int stages = epi_bytes + stage_bytes <= budget ? (int)((budget - epi_bytes) / stage_bytes) : 1;
-    if (stages > TC_MAX_STAGES) stages = TC_MAX_STAGES;
-    if (stages > min_chunks) stages = min_chunks;
-    ta.stages = stages;
-    const size_t smem = (size_t)stages * stage_bytes + epi_bytes + 1024;
-    CK(launch(k_gemm_tc<Epi>, dim3(splits, tiles, m_blocks), TC_THREADS, smem, s, a0, a1, mx, ta, ep));
-    e->launches++;
+    const TcCtx cx{wsp<float>(e, L.tc_partial), wsp<int32_t>(e, L.tc_counters), wsp<int32_t>(e, L.flag),
+                   env_off("VUIB_TRACE") ? wsp<unsigned long long>(e, L.trace) : nullptr, &e->num_sms, e->spin_limit,
+                   &e->launches};
+    CK(tc_gemm_launch(cx, a0, a1, X, K, M, K, units, row_off, ep, s));
     return VUIB_OK;
 }
 

@@ -16,7 +16,6 @@ this library's own kernels); pass it, or any object with ``decode(codes_bqt)`` a
 from __future__ import annotations
 
 import ctypes as C
-from collections import deque
 from collections.abc import Iterator
 from dataclasses import dataclass
 from types import SimpleNamespace
@@ -26,6 +25,8 @@ from torch import Tensor
 
 from . import _lib
 from .model import VuiB200
+from .registry import load_model
+from .slots import SlotEngine, _get_bucket, _make_buckets  # noqa: F401 - the bucket helpers keep their old import path
 from .text import chunk_text, simple_clean
 
 FRAME_RATE = 12.5  # codec frames per second (src/vui/qwen_codec.py:27-29)
@@ -102,23 +103,6 @@ class _ActiveSlot:
     seq_offset: int = 0
 
 
-def _make_buckets(max_bs: int) -> list[int]:
-    out, b = [], 1
-    while b < max_bs:
-        out.append(b)
-        b *= 2
-    if not out or out[-1] != max_bs:
-        out.append(max_bs)
-    return out
-
-
-def _get_bucket(n: int, buckets: list[int]) -> int:
-    for b in buckets:
-        if n <= b:
-            return b
-    return buckets[-1]
-
-
 class Row:
     """A single conversation slot: index into the shared KV cache, the
     end-of-prompt offset for rewind, and the speaker token(s) from prefill."""
@@ -177,10 +161,11 @@ class Row:
         self.close()
 
 
-class Engine:
+class Engine(SlotEngine):
     """Streaming (max_rows=1) and batched (max_rows=N) inference over one model."""
 
     NAMES = {"vui-nano": "vui-nano.safetensors"}
+    _ROW = Row
 
     def __init__(self, name: str = "vui-nano", *, model: VuiB200 | None = None, codec=None,
                  max_rows: int = 1, max_seq: int | None = None, codec_dtype: torch.dtype = torch.float32,
@@ -188,12 +173,14 @@ class Engine:
         if not torch.cuda.is_available():
             raise RuntimeError("vui_b200.Engine needs a CUDA device (sm_100a); there is no CPU path")
         if model is None:
-            model = VuiB200.from_checkpoint(self.NAMES.get(name, name))
+            model = load_model(self.NAMES.get(name, name))
+            if not isinstance(model, VuiB200):
+                raise ValueError(f"'{name}' is not a speech model; open it with vui_b200.open_engine")
         self.model = model
         self.codec = codec
         self.overlap_codec = False   # True: Row.stream decodes frame k's audio beside the generation of frame k + 1
         self._codec_stream = None
-        self.max_rows = max_rows
+        self._init_slots(max_rows)
         self.vocoder_ctx = vocoder_ctx
         self.device = model.device
         self.dtype = model.dtype
@@ -220,22 +207,12 @@ class Engine:
         self._capture_stream = None
         self._sampling_key = None
         self._setup_native()
-        self._free: set[int] = set(range(max_rows))
-        self._rows: dict[int, Row] = {}
         self._rep_window_cur = 0
 
     # ------------------------------------------------------------------ setup
-    def _ck(self, code: int) -> None:
-        _lib.check(self._handle, code)
-
-    @property
-    def _stream(self):
-        return C.c_void_p(torch.cuda.current_stream(self.device).cuda_stream)
-
     def _setup_native(self) -> None:
         s, dev = self.model.shape, self.device
         n_slots = self.max_rows + 1  # spare slot: target of padded rows (engine.py:380-387)
-        self._pad_slot = self.max_rows
         cfg = _lib.VuibConfig(
             s.d_model, s.n_layers, s.n_heads, s.n_kv_heads, s.head_dim, s.intermediate_size,
             s.n_quantizers, s.codebook_size, s.rq_d_model, s.rq_n_layers, s.rq_n_heads, s.rq_ffn,
@@ -294,7 +271,6 @@ class Engine:
         self._ck(self._lib.vuib_set_stats(self._handle, C.c_void_p(self._g_cb0_stats.data_ptr())))
         self._g_slot_idx = torch.arange(N, device=dev, dtype=torch.int32)
         self._g_seq_inc = torch.ones(N, device=dev, dtype=torch.int32)
-        self._buckets = _make_buckets(N)
         # pinned landing zone for the one read-back per frame
         self._h_codes = torch.zeros(N, self.Q, dtype=torch.long).pin_memory()
         self._h_eos = torch.zeros(N, dtype=torch.float32).pin_memory()
@@ -302,26 +278,11 @@ class Engine:
         self._done = torch.cuda.Event()
         self._set_sampling(1.0, 1, 1, 1.0, 0, 0)
 
-    def __del__(self):
-        try:
-            if self._handle:
-                self._lib.vuib_destroy(self._handle)
-                self._handle = C.c_void_p()
-        except Exception:
-            pass
-
     @classmethod
     def from_checkpoint(cls, checkpoint_path: str, *, max_rows: int = 1, max_seq: int | None = None,
                         codec_dtype: torch.dtype = torch.float32, vocoder_ctx: int = 25) -> "Engine":
         return cls(checkpoint_path, max_rows=max_rows, max_seq=max_seq, codec_dtype=codec_dtype,
                    vocoder_ctx=vocoder_ctx)
-
-    def launch_count(self) -> int:
-        return int(self._lib.vuib_launch_count(self._handle))
-
-    def check_device(self) -> None:
-        """Raise if a kernel saw a slot, position or code out of range."""
-        self._ck(self._lib.vuib_check_device_flag(self._handle, self._stream))
 
     # --------------------------------------------------------------- sampling
     def _set_sampling(self, temperature, top_k_cb0, top_k_rq, rep_penalty, rep_window, n_codebooks) -> None:
@@ -378,41 +339,22 @@ class Engine:
         g = self._graphs.get(B)
         if g is not None:
             return g
-        # One warm-up outside capture loads the kernels; it runs on the spare slot
-        # with the length frozen, and the sampler state it touched is put back.
-        saved = (self._g_slot_idx.clone(), self._g_seq_inc.clone(), self._g_codes_in.clone(),
-                 self.seq_lens.clone(), self._ws.clone())
-        self._g_slot_idx.fill_(self._pad_slot)
-        self._g_seq_inc.zero_()
+        # the warm-up run uses code 0 everywhere; the codes and the sampler state it touched are put back
+        def call():
+            self._frame_call(B)
+
+        codes = self._g_codes_in.clone()
         self._g_codes_in.zero_()
-        self.seq_lens[self._pad_slot] = 0
-        torch.cuda.synchronize(self.device)
-        side = torch.cuda.Stream(self.device)
-        side.wait_stream(torch.cuda.current_stream(self.device))
-        with torch.cuda.stream(side):
-            self._frame_call(B)
-        torch.cuda.current_stream(self.device).wait_stream(side)
-        torch.cuda.synchronize(self.device)
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._frame_call(B)
-        torch.cuda.synchronize(self.device)
-        self._g_slot_idx.copy_(saved[0])
-        self._g_seq_inc.copy_(saved[1])
-        self._g_codes_in.copy_(saved[2])
-        self.seq_lens.copy_(saved[3])
-        self._ws.copy_(saved[4])
+        g = self._capture_graph(call, [self._g_codes_in, self._ws])
+        self._g_codes_in.copy_(codes)
         self._graphs[B] = g
         return g
 
     def _frame_step(self, B_active: int):
         """Replay one whole frame for the first B_active rows of the static
         buffers (padded to the bucket with rows aimed at the spare slot)."""
-        B = _get_bucket(B_active, self._buckets)
-        g = self._frame_graph(B)
-        if B_active < B:
-            self._g_slot_idx[B_active:B].fill_(self._pad_slot)
-            self._g_seq_inc[B_active:B].zero_()
+        g = self._frame_graph(_get_bucket(B_active, self._buckets))
+        self._pad_to_bucket(B_active)
         g.replay()
 
     def _frame_host(self, B_active: int, h_codes_in: Tensor | None = None):
@@ -433,9 +375,7 @@ class Engine:
                 P(self._g_hidden_out), P(self._g_cb0_out), P(self._g_eos_out), P(self._g_eos_prob),
                 C.c_void_p(self._capture_stream.cuda_stream)))
             self._host_frames.add((B, with_in))
-        if B_active < B:
-            self._g_slot_idx[B_active:B].fill_(self._pad_slot)
-            self._g_seq_inc[B_active:B].zero_()
+        self._pad_to_bucket(B_active)
         src = None
         if with_in:
             if h_codes_in.dtype != torch.long or not h_codes_in.is_contiguous() or h_codes_in.is_cuda:
@@ -478,30 +418,10 @@ class Engine:
         mk = getattr(self.codec, "new_ctx", None)
         return mk() if mk else None
 
-    def new_row(self) -> Row:
-        if not self._free:
-            raise RuntimeError(f"No free rows (max_rows={self.max_rows} all in use)")
-        idx = min(self._free)
-        self._free.remove(idx)
-        row = Row(self, idx)
-        self._rows[idx] = row
-        self.seq_lens[idx] = 0
-        return row
-
     def _release_row(self, row: Row) -> None:
-        self._rows.pop(row.idx, None)
-        self._free.add(row.idx)
+        super()._release_row(row)
         if row._codec_ctx is not None:
             row._codec_ctx.reset()
-
-    def reset(self) -> None:
-        for row in list(self._rows.values()):
-            row.close()
-        self.seq_lens.zero_()
-
-    def _rewind_row(self, row: Row, offset: int) -> int:
-        self.seq_lens[row.idx] = offset
-        return offset
 
     def set_conditioning(self, *, sq_scores=None, wps_score: float = 0.0) -> None:
         """SQ / WPS conditioning bias added to text embeddings (Vui.set_cond_bias,
@@ -519,55 +439,26 @@ class Engine:
     def _prefill_many(self, items: list[tuple[Row, Tensor]]) -> list[Tensor]:
         """Prefill several (row, emb (T_i, d)) pairs in as few calls as fit
         max_prefill_rows.  Returns each row's final-norm output (T_i, d)."""
-        outs = []
-        pend: list[tuple[int, int, Tensor]] = []  # slot, offset, emb
+        items = [(row, emb.reshape(-1, self.D)) for row, emb in items]
+        parts: list[list[Tensor]] = [[] for _ in items]
 
-        def flush():
-            if not pend:
-                return
-            emb = torch.cat([e for _, _, e in pend], dim=0).to(self.dtype).contiguous()
-            slot = torch.cat([torch.full((e.shape[0],), s_, dtype=torch.int32) for s_, _, e in pend])
-            pos = torch.cat([torch.arange(o, o + e.shape[0], dtype=torch.int32) for _, o, e in pend])
+        def run(pend):
+            emb = torch.cat([e for _, _, e, _ in pend], dim=0).to(self.dtype).contiguous()
+            slot = torch.cat([torch.full((e.shape[0],), s_, dtype=torch.int32) for s_, _, e, _ in pend])
+            pos = torch.cat([torch.arange(o, o + e.shape[0], dtype=torch.int32) for _, o, e, _ in pend])
             slot, pos = slot.to(self.device), pos.to(self.device)
             out = torch.empty_like(emb)
             P = lambda t: C.c_void_p(t.data_ptr())  # noqa: E731
             self._ck(self._lib.vuib_prefill(self._handle, emb.shape[0], P(slot), P(pos), P(emb), P(out),
                                             self._stream))
             i = 0
-            for s_, _, e in pend:
-                outs.append(out[i:i + e.shape[0]])
+            for s_, _, e, k in pend:
+                parts[k].append(out[i:i + e.shape[0]])
                 self.seq_lens[s_] += e.shape[0]
                 i += e.shape[0]
-            pend.clear()
 
-        offsets = {}
-        for row, emb in items:
-            emb = emb.reshape(-1, self.D)
-            off = offsets.get(row.idx, row.offset)
-            if off + emb.shape[0] > self.max_seq:
-                raise RuntimeError(f"prefill of {emb.shape[0]} positions overflows max_seq={self.max_seq}")
-            # a segment longer than one call is cut; a slot may appear several times in a call (its rows
-            # carry consecutive positions, and every row's K/V is in the cache before any row attends)
-            start = 0
-            while start < emb.shape[0]:
-                room = self.max_prefill_rows - sum(e.shape[0] for _, _, e in pend)
-                if room == 0:
-                    flush()
-                    room = self.max_prefill_rows
-                n = min(room, emb.shape[0] - start)
-                pend.append((row.idx, off + start, emb[start:start + n]))
-                start += n
-            offsets[row.idx] = off + emb.shape[0]
-        flush()
-        # stitch cut segments back together per input item
-        res, k = [], 0
-        for row, emb in items:
-            T, parts = emb.reshape(-1, self.D).shape[0], []
-            while sum(p.shape[0] for p in parts) < T:
-                parts.append(outs[k])
-                k += 1
-            res.append(torch.cat(parts, dim=0) if len(parts) > 1 else parts[0])
-        return res
+        self._pack_rows(items, run)
+        return [torch.cat(p, dim=0) if len(p) > 1 else p[0] for p in parts]
 
     def _prefill_emb(self, row: Row, emb: Tensor) -> Tensor:
         """Write (1, T, d) embeddings into the row's slot at its current offset;
@@ -913,9 +804,6 @@ class Engine:
         min_frames = int(cfg.min_secs * FRAME_RATE)
         max_seq = self.max_seq - 10
         bufs: list[list[Tensor]] = [[] for _ in requests]
-        pending: deque[int] = deque(range(len(requests)))
-        active: dict[int, _ActiveSlot] = {}
-        free_slots = set(range(self.max_rows))
         last_codes: dict[int, Tensor] = {}
         self._apply_cfg(cfg)
         # continuous batching keeps penalty counts without a window (engine.py:606-616)
@@ -938,12 +826,10 @@ class Engine:
             info.seq_offset = row.offset
             return True
 
-        def backfill() -> None:
-            while pending and free_slots:
-                ri = pending.popleft()
+        def admit(batch) -> dict[int, _ActiveSlot]:
+            started = {}
+            for ri, slot in batch:
                 req = requests[ri]
-                slot = min(free_slots)
-                free_slots.remove(slot)
                 self.seq_lens[slot] = 0
                 self._rep_reset(slot=slot)
                 row = Row(self, slot)
@@ -954,15 +840,11 @@ class Engine:
                 chunks = chunk_text(req.text, min_words=cfg.chunk_words, sentence_only=cfg.sentence_only,
                                     single_speaker=(row._spk_token_2 is None))
                 info = _ActiveSlot(row=row, request_idx=ri, chunks=chunks)
-                if not chunks or not advance(info):
-                    self._rows.pop(slot, None)
-                    free_slots.add(slot)
-                    continue
-                active[slot] = info
+                if chunks and advance(info):
+                    started[slot] = info
+            return started
 
-        backfill()
-        while active:
-            slots = sorted(active)
+        def step(slots, infos) -> list[int]:
             B = len(slots)
             for qi, s_ in enumerate(slots):
                 self._set_codes_in(qi, last_codes[s_])
@@ -972,8 +854,7 @@ class Engine:
             h_codes, h_eos = self._read_frame(B)
             h_codes = h_codes.clone()
             done = []
-            for qi, s_ in enumerate(slots):
-                info = active[s_]
+            for qi, (s_, info) in enumerate(zip(slots, infos)):
                 info.seq_offset += 1
                 if info.frame_count >= max_frames or info.seq_offset >= max_seq:
                     done.append(s_)
@@ -988,11 +869,9 @@ class Engine:
                 bufs[info.request_idx].append(h_codes[qi][None])
                 info.frame_count += 1
                 info.turn_count += 1
-            for s_ in done:
-                info = active.pop(s_)
-                self._rows.pop(s_, None)
-                free_slots.add(s_)
-            backfill()
+            return done
+
+        self._run_continuous(len(requests), admit, step)
         return [torch.cat(b, dim=0) if b else torch.zeros(0, self.Q, dtype=torch.long) for b in bufs]
 
     # -------------------------------------------------------------- streaming

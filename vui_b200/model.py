@@ -115,6 +115,8 @@ class VuiB200(torch.nn.Module):
     """Parameter container.  ``sd`` maps reference state-dict names to tensors;
     they are moved to ``device`` as bf16 and kept contiguous."""
 
+    architecture = "Vui"
+
     def __init__(self, shape: VuiShape, sd: dict[str, Tensor], device="cuda", tokenizer=None):
         super().__init__()
         self.shape = shape
