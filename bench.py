@@ -23,6 +23,10 @@ Under torchrun (N > 1) every rank is an independent replica with its own streams
 on its own GPU; there is no data-path collective, the process group only aligns
 the timed window and takes the max time over ranks.
 
+`--token-model` times the token model's prefill and decode at several sizes beside the speech backbone at equal size
+(a JSON line of its own, nothing of the default workload); `--profile-token-model B` runs one decode step of B rows and one
+prefill of both models kernel by kernel and exits.
+
 `--impl reference` times the CPU restatement of the reference's PyTorch path
 (oracle/, fp32, all host threads) on the same metric.  `--profile-frames N` runs N
 frames kernel by kernel (no graph) and exits: the command the ncu summaries under
@@ -642,6 +646,237 @@ def profile_frames(model, dev, n, B, prompt_len):
                       "launches_per_frame": (eng.launch_count() - before) // max(n, 1)}), flush=True)
 
 
+# ---------------------------------------------------------------------------- token models
+# width, layers, heads, MLP; the speech backbone takes the same figures (8-row GQA), the token model the latent sizes
+LM_SIZES = {
+    "512x12": dict(width=512, layers=12, heads=8, ff=1536, dim=64, rot_dim=32, vdim=64, q_rank=256, kv_rank=128),
+    "1024x24": dict(width=1024, layers=24, heads=16, ff=3072, dim=64, rot_dim=32, vdim=64, q_rank=512, kv_rank=256),
+    "1536x24": dict(width=1536, layers=24, heads=24, ff=3072, dim=64, rot_dim=32, vdim=64, q_rank=768, kv_rank=256),
+    # layers of a larger model; the speech engine has no such size
+    "4096x8": dict(width=4096, layers=8, heads=32, ff=14336, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512),
+}
+LM_VOCAB = 2048
+
+
+def lm_model(size, dev):
+    from vui_b200.token_lm import ClampedGLU, LatentMixer, LayerSpec, TokenLMConfig, Vidotar
+
+    m = LatentMixer(heads=size["heads"], dim=size["dim"], rot_dim=size["rot_dim"], vdim=size["vdim"], q_rank=size["q_rank"],
+                    kv_rank=size["kv_rank"], scale=(size["dim"] + size["rot_dim"]) ** -0.5, rot_base=10000.0,
+                    rot_dims=size["rot_dim"])
+    layers = (LayerSpec(m, ClampedGLU(ff=size["ff"], limit=7.0)),) * size["layers"]
+    return Vidotar.random_init(TokenLMConfig(LM_VOCAB, size["width"], 1e-5, 1.0, layers), seed=0, device=dev)
+
+
+def backbone_model(size, dev):
+    from vui_b200 import VuiB200, VuiShape
+
+    shape = VuiShape(d_model=size["width"], n_layers=size["layers"], n_heads=size["heads"], n_kv_heads=size["heads"] // 2,
+                     intermediate_size=size["ff"], vocab_size=LM_VOCAB, rq_n_layers=1)
+    return VuiB200.random_init(shape, seed=0, device=dev)
+
+
+class ColdTimer:
+    """Median device time of a call with L2 written over before each run."""
+
+    def __init__(self, dev, n=15):
+        import torch
+
+        self.torch, self.dev, self.n = torch, dev, n
+        self.junk = torch.empty(512 << 20, dtype=torch.uint8, device=dev)
+
+    def __call__(self, fn, before=None):
+        torch = self.torch
+        for _ in range(3):
+            if before:
+                before()
+            fn()
+        times = []
+        for _ in range(self.n):
+            if before:
+                before()
+            self.junk.fill_(1)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize(self.dev)
+            self.junk[: 256 << 20].fill_(2)   # keeps the device busy while the host enqueues
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize(self.dev)
+            times.append(a.elapsed_time(b))
+        return statistics.median(times)
+
+
+class LmBench:
+    """The token model's engine at fixed context, and what its decode and prefill move and multiply."""
+
+    def __init__(self, size, dev, rows, ctx, prefill_rows):
+        import torch
+
+        from vui_b200 import TokenEngine
+
+        self.size, self.ctx = size, ctx
+        self.model = lm_model(size, dev)
+        self.eng = TokenEngine(model=self.model, max_rows=rows, max_seq=2048, max_prefill_rows=prefill_rows)
+        for c in self.eng.cache:
+            c[..., : size["kv_rank"]].normal_()
+        self.torch = torch
+
+    def rewind(self, n):
+        self.eng.seq_lens.fill_(n)
+        self.eng._len = [n] * (self.eng.max_rows + 1)
+
+    def decode_graph(self, B):
+        self.eng._aim(list(range(B)))
+        self.rewind(self.ctx)
+        return self.eng._step_graph(B, False)
+
+    def decode_call(self, B):
+        self.eng._aim(list(range(B)))
+        self.eng._step_call(B, False)
+
+    def prefill(self, n_seq, n_tok):
+        """n_seq prompts of n_tok tokens, logits of each last token."""
+        self.rewind(0)
+        rows = [type("R", (), {"idx": i, "offset": 0})() for i in range(n_seq)]
+        ids = self.torch.arange(n_tok) % LM_VOCAB
+        out = self.torch.empty(n_seq, LM_VOCAB, device=self.eng.device)
+        portions = [(r, ids, [n_tok - 1], i) for i, r in enumerate(rows)]
+        return lambda: self.eng._prefill(portions, out)
+
+    def decode_bytes(self, B):
+        z = self.size
+        return self.model.weight_bytes_per_step() + B * z["layers"] * 2 * (self.ctx + 1) * (z["kv_rank"] + z["rot_dim"])
+
+    def prefill_flops(self, n_seq, n_tok):
+        z = self.size
+        per_tok = 2 * (sum(t.numel() for k, t in self.model.sd.items() if t.dim() == 2 and k not in ("embed", "head")))
+        attn = z["layers"] * z["heads"] * n_tok * (n_tok + 1) * (z["dim"] + z["rot_dim"] + z["vdim"])
+        return n_seq * (n_tok * per_tok + attn)
+
+
+class BackboneBench:
+    """The speech backbone (embedding, layers, heads; no depth transformer) at the same sizes."""
+
+    def __init__(self, size, dev, rows, ctx, prefill_rows):
+        import torch
+
+        from vui_b200 import Engine
+
+        self.size, self.ctx, self.torch = size, ctx, torch
+        self.model = backbone_model(size, dev)
+        self.eng = Engine(model=self.model, max_rows=rows, max_seq=2048, max_prefill_rows=prefill_rows)
+        self.eng._kv.normal_()
+
+    def decode_call(self, B):
+        import ctypes as C
+
+        e = self.eng
+        P = lambda t: C.c_void_p(t.data_ptr())  # noqa: E731
+        e._ck(e._lib.vuib_backbone_step(e._handle, B, P(e._g_slot_idx), P(e._g_seq_inc), P(e._g_codes_in), P(e._g_hidden_out),
+                                        P(e._g_cb0_out), P(e._g_eos_out), e._stream))
+
+    def rewind(self, n):
+        self.eng.seq_lens.fill_(n)
+
+    def decode_graph(self, B):
+        e = self.eng
+        e._g_slot_idx[:B] = self.torch.arange(B, device=e.device, dtype=self.torch.int32)
+        e._g_seq_inc.fill_(1)
+        self.rewind(self.ctx)
+        return e._capture_graph(lambda: self.decode_call(B), [e._g_codes_in])
+
+    def prefill(self, n_seq, n_tok):
+        import ctypes as C
+
+        e, torch = self.eng, self.torch
+        n = n_seq * n_tok
+        emb = torch.randn(n, self.size["width"], device=e.device).to(e.dtype)
+        slot = torch.arange(n_seq, device=e.device, dtype=torch.int32).repeat_interleave(n_tok)
+        pos = torch.arange(n_tok, device=e.device, dtype=torch.int32).repeat(n_seq)
+        out = torch.empty_like(emb)
+        P = lambda t: C.c_void_p(t.data_ptr())  # noqa: E731
+        return lambda: e._ck(e._lib.vuib_prefill(e._handle, n, P(slot), P(pos), P(emb), P(out), e._stream))
+
+    def layer_params(self):
+        return sum(t.numel() for k, t in self.model.sd.items() if k.startswith("decoder.blocks.") and t.dim() == 2)
+
+    def decode_bytes(self, B):
+        z = self.size
+        return 2 * (self.layer_params() + LM_VOCAB * z["width"]) + B * z["layers"] * 2 * (self.ctx + 1) * z["heads"] * 64
+
+    def prefill_flops(self, n_seq, n_tok):
+        z = self.size
+        return n_seq * (n_tok * 2 * self.layer_params() + z["layers"] * z["heads"] * n_tok * (n_tok + 1) * 128)
+
+
+def token_model_bench(args):
+    import torch
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm, kind = measured_hbm_peak()
+    tf = None
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(p):
+        with open(p) as f:
+            tf = float(json.load(f)["bf16_tflops"])
+    tf = tf or 1590.0
+    timer = ColdTimer(dev)
+    ctx, prefills = 512, ((16, 256), (2, 2048))
+    sampler = ClockSampler(dev.index or 0)
+    sampler.start()
+    res = {}
+    for name, size in LM_SIZES.items():
+        if args.token_sizes and name not in args.token_sizes.split(","):
+            continue
+        res[name] = {}
+        for label, cls in (("vidotar", LmBench), ("vui_backbone", BackboneBench)):
+            if label == "vui_backbone" and size["width"] > 1536:
+                continue
+            b = cls(size, dev, 64, ctx, 4096)
+            r = {"decode": {}, "prefill": {}}
+            for B in (1, 4, 16, 64):
+                before = b.eng.launch_count()
+                g = b.decode_graph(B)
+                launches = (b.eng.launch_count() - before) // 2
+                ms = timer(g.replay, before=lambda: b.rewind(ctx))
+                r["decode"][B] = {"ms": round(ms, 4), "tokens_per_s": round(B / ms * 1e3), "launches": launches,
+                                  "hbm_frac": round(b.decode_bytes(B) / ms / 1e6 / hbm, 4)}
+            for n_seq, n_tok in prefills:
+                fn = b.prefill(n_seq, n_tok)
+                ms = timer(fn, before=lambda: b.rewind(0))
+                r["prefill"][f"{n_seq}x{n_tok}"] = {"ms": round(ms, 3), "tokens_per_s": round(n_seq * n_tok / ms * 1e3),
+                                                    "bf16_frac": round(b.prefill_flops(n_seq, n_tok) / ms / 1e9 / tf, 4)}
+            b.eng.check_device()
+            res[name][label] = r
+            del b, g, fn
+            torch.cuda.empty_cache()
+    print(json.dumps({
+        "metric": "token model prefill and decode", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16",
+        "config": {"context": ctx, "vocab": LM_VOCAB, "l2": "written over (256 MB) before every timed call",
+                   "timing": "CUDA events, median of 15 calls", "hbm_gbs": hbm, "bf16_tflops": tf, "peaks": kind},
+        "sizes": res, "clocks": sampler.stop()}), flush=True)
+
+
+def profile_token_model(args):
+    """One eager decode step of B rows and one prefill of 16 x 256 of both models at 1024x24 (4 layers of it)."""
+    import torch
+
+    dev = torch.device("cuda", 0)
+    size = dict(LM_SIZES["1024x24"], layers=2)
+    for cls in (LmBench, BackboneBench):
+        b = cls(size, dev, max(args.profile_token_model, 16), 512, 4096)
+        B = args.profile_token_model
+        for _ in range(2):
+            b.rewind(512)
+            b.decode_call(B)
+        b.prefill(16, 256)()
+        torch.cuda.synchronize(dev)
+        b.eng.check_device()
+        print(json.dumps({"profile": cls.__name__, "launches": b.eng.launch_count()}), flush=True)
+
+
 def run_b200(args):
     import torch
     import torch.distributed as dist
@@ -795,7 +1030,16 @@ def main():
     ap.add_argument("--profile-frames", type=int, default=0, help="run N frames without a graph and exit (for ncu)")
     ap.add_argument("--profile-codec", type=int, default=0, help="run N streamed codec frames without a graph and exit")
     ap.add_argument("--profile-encoder", type=int, default=0, help="run N codec-encoder calls on a 10 s buffer and exit")
+    ap.add_argument("--token-model", action="store_true", help="token model prefill / decode beside the speech backbone, and exit")
+    ap.add_argument("--token-sizes", default="", help="with --token-model: sizes to run, separated by commas")
+    ap.add_argument("--profile-token-model", type=int, default=0, metavar="B", help="one decode step of B rows and one prefill, and exit")
     args = ap.parse_args()
+    if args.token_model:
+        token_model_bench(args)
+        return
+    if args.profile_token_model:
+        profile_token_model(args)
+        return
     if args.warmup < 3:
         args.warmup = 3
     if args.impl == "reference":

@@ -209,7 +209,7 @@ cudaError_t allow_smem(const void* kern, size_t bytes) {
     if (err != cudaSuccess) return err;
     std::lock_guard<std::mutex> lock(mu);
     size_t& h = have[{dev, kern}];
-    if (bytes <= 48 * 1024 || bytes <= h) return cudaSuccess;
+    if (bytes <= 32 * 1024 || bytes <= h) return cudaSuccess;   // static shared memory counts towards the 48 KB default
     err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
     if (err == cudaSuccess) h = bytes;
     return err;
