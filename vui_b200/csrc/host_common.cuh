@@ -41,21 +41,38 @@ static void prefer_max_smem(const void* kern) {
         cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
 }
 
+// `cluster_x` > 1 groups that many consecutive CTAs of the grid's x dimension into a cluster.
 template <class... KArgs, class... Args>
-static cudaError_t launch(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s,
-                          Args... args) {
+static cudaError_t launch_cl(void (*kern)(KArgs...), dim3 grid, int cluster_x, dim3 block, size_t smem, cudaStream_t s,
+                             Args... args) {
     prefer_max_smem(reinterpret_cast<const void*>(kern));
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
     cfg.dynamicSmemBytes = smem;
     cfg.stream = s;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (cluster_x > 1) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = cluster_x;
+        attr[n].val.clusterDim.y = 1;
+        attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    if (pdl_enabled()) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
     cfg.attrs = attr;
-    cfg.numAttrs = pdl_enabled() ? 1 : 0;
+    cfg.numAttrs = n;
     return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
+}
+
+template <class... KArgs, class... Args>
+static cudaError_t launch(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
+    return launch_cl(kern, grid, 1, block, smem, s, args...);
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
@@ -120,10 +137,16 @@ static inline size_t tc_partial_bytes(size_t max_rows) {
     return (size_t)(TC_PARTIAL_TILES + 80) * TC_TILE_N * (max_rows < 256 ? ((max_rows + 15) / 16) * 16 : 256) * 4;
 }
 
+// Epilogue staging per activation row: what the functor says, TC_EPI_BYTES_PER_M when it does not.
+template <class Epi>
+static auto tc_stage_bytes(const Epi& ep, int) -> decltype(ep.stage_bytes_per_row()) { return ep.stage_bytes_per_row(); }
+template <class Epi>
+static size_t tc_stage_bytes(const Epi&, long) { return TC_EPI_BYTES_PER_M; }
+
 // D = W X^T over all M rows in blocks of <= 256, epilogue ep (see tc_gemm.cuh).
 //  units: weight rows (N, multiple of 128) or, for the paired SwiGLU form, hidden units (multiple of 64).
 //  x_split_tile / x_split_row: weight tiles from x_split_tile on multiply the M rows that start x_split_row rows
-//  further down in X (two inputs of one launch); x_rows = rows of X the map may cover.
+//  further down in X (two inputs of one launch).
 template <class Epi>
 static cudaError_t tc_gemm_launch(const TcCtx& cx, const CUtensorMap& a0, const CUtensorMap& a1, const bf16* X, int ldx,
                                   int M, int K, int units, int row_off, const Epi& ep, cudaStream_t s,
@@ -182,7 +205,7 @@ static cudaError_t tc_gemm_launch(const TcCtx& cx, const CUtensorMap& a0, const 
     ta.x_split_row = x_split_row;
     const int min_chunks = chunks_total / splits;  // the shortest split
     const size_t stage_bytes = TC_TILE_N * TC_KCHUNK * 2 + ((Mpad * TC_KCHUNK * 2 + 1023) & ~1023);
-    const size_t epi_bytes = Epi::STAGED ? (size_t)Mpad * TC_EPI_BYTES_PER_M : 0;
+    const size_t epi_bytes = Epi::STAGED ? (size_t)Mpad * tc_stage_bytes(ep, 0) : 0;
     // two CTAs per SM when split (all CTAs of the grid must be resident), the whole SM otherwise
     const size_t budget = (splits > 1 ? 100 : 200) * 1024;
     int stages = epi_bytes + stage_bytes <= budget ? (int)((budget - epi_bytes) / stage_bytes) : 1;

@@ -4,8 +4,9 @@
 // Absorbed form (decode, short portions).  With the key matrix folded into the query projection at load time, a
 // query head is a vector over the whole cached row, score = scale * q_h . row, and its output before the value
 // matrix is sum_j p_j c_j.  The 16 rows of an MMA tile are the HEADS of one query row, so a key tile is read once
-// for all of them.  k_latent_attn: CTA = (split of the keys, 16 heads x a block of columns, query row); the partial
-// sums meet in k_latent_out, which also applies the value matrix and the output gate.
+// for all of them.  k_latent_attn (bf16): a cluster of CTAs per query row splits the keys and merges through distributed
+// shared memory; for a few rows it also applies the value matrix and the output gate, for more k_latent_value does.
+// k_latent_attn_f32 leaves partial sums that meet in k_latent_out.
 //
 // Expanded form (prefill).  Keys and values of a call's sequences are expanded once per layer by a GEMM, and
 // k_latent_prefill walks query tile x key tile per head, as k_prefill_attn (prefill_attn.cuh) does.
@@ -53,17 +54,33 @@ __device__ __forceinline__ void split_bf16x2(float p0, float p1, uint32_t& hi, u
     lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
+// n / d for the small indices of the copy loops: d's reciprocal rounded up, exact while n * d < 2^32.
+struct FastDiv {
+    uint32_t d, mul;
+    FastDiv() = default;
+    explicit FastDiv(int v) : d((uint32_t)v), mul((uint32_t)(((1ull << 32) + v - 1) / v)) {}   // v >= 2
+    __device__ __forceinline__ int div(int n) const { return (int)__umulhi((uint32_t)n, mul); }
+};
+
 struct LatentAttnArgs {
     const void* q;            // (M, H, Dp) T
     const void* cache;        // (n_slots, max_seq, Dp) T of this layer
     const int32_t* row_slot;
     const int32_t* row_pos;
-    float* part;              // (M, S, H, Rp)
-    float* ml;                // (M, S, H, 2): running maximum and sum
-    int H, Rp, Dp, max_seq, S;
-    int col_blocks;           // grid.y = head groups of 16 x column blocks
+    int H, Rp, Dp, max_seq;
     int nbuf;                 // key tiles in shared memory (1 or 2)
     float scale;
+    FastDiv row_vecs;         // Dp / 8
+    // bf16: value matrix and gate (fused), or the latent sums (M, H, Rp)
+    const bf16* wuv;          // (H, vdim, Rp)
+    const bf16* gate;         // (M, ldgate)
+    bf16* out;                // fused: (M, ldo) gated values; else the latent sums
+    int ldgate, ldo, vdim;
+    // fp32: partial sums of the splits
+    float* part;              // (M, S, H, Rp)
+    float* ml;                // (M, S, H, 2): running maximum and sum
+    int S;
+    int col_blocks;           // grid.y = head groups of 16 x column blocks
 };
 
 // How the keys of a row of `len` positions are dealt to S splits in tiles of `keys`: tiles per split, splits in use.
@@ -73,57 +90,88 @@ __device__ __forceinline__ void latent_splits(int len, int keys, int S, int& tps
     ns = (nt + tps - 1) / tps;
 }
 
-static inline size_t latent_attn_smem(int Dp, int nbuf) {
-    return (size_t)(16 + nbuf * LA_KEYS) * (Dp + 8) * 2 + 16 * (LA_KEYS + 4) * 4 + 2 * 16 * (LA_KEYS + 8) * 2 + 16 * 4;
+constexpr int LA_MAX_CL = 8;      // CTAs (key splits) of a row's cluster
+
+static inline size_t latent_attn_smem(int Dp, int Rp, int nbuf, int fuse_heads = 0) {
+    const size_t keys = (size_t)nbuf * LA_KEYS * (Dp + 8) * 2, sums = (size_t)16 * (Rp + 4) * 4;   // share their space
+    return (size_t)16 * (Dp + 8) * 2 + (keys > sums ? keys : sums) + 16 * (LA_KEYS + 4) * 4 + 2 * 16 * (LA_KEYS + 8) * 2 +
+           16 * 4 + 16 * 8 + (size_t)fuse_heads * Rp * 4;
 }
 
-template <int NT>  // n-tiles (8 columns) per warp; a CTA covers NT * 64 columns of c
-static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArgs a) {
+__device__ __forceinline__ uint32_t cluster_addr(const void* p, int rank) {
+    uint32_t ra;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(rank));
+    return ra;
+}
+__device__ __forceinline__ float ld_cluster(uint32_t a) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
+    return v;
+}
+__device__ __forceinline__ float2 ld_cluster2(uint32_t a) {
+    float2 v;
+    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(a) : "memory");
+    return v;
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
+// One cluster of CL CTAs per (query row, 16 heads): CTA = a split of the keys.  The CTAs leave their partial sums in
+// shared memory; each then merges 16 / CL heads over the cluster in split order, and either writes the latent sums or
+// (FUSE_V, few rows) multiplies them with its heads' value matrices and gates the result.
+template <int NT, bool FUSE_V>  // n-tiles (8 columns of c) per warp
+static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArgs a, int CL) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     pdl_trigger();
-    const int ld = a.Dp + 8;
+    const int ld = a.Dp + 8, lds = a.Rp + 4;
+    constexpr int SP = LA_KEYS + 4, PP = LA_KEYS + 8;
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);
     bf16* Ks = Qs + 16 * ld;
-    float* Ss = reinterpret_cast<float*>(Ks + (size_t)a.nbuf * LA_KEYS * ld);
-    bf16* Ph = reinterpret_cast<bf16*>(Ss + 16 * (LA_KEYS + 4));
-    bf16* Pl = Ph + 16 * (LA_KEYS + 8);
-    float* corr_s = reinterpret_cast<float*>(Pl + 16 * (LA_KEYS + 8));
-    constexpr int SP = LA_KEYS + 4, PP = LA_KEYS + 8;
+    float* Os = reinterpret_cast<float*>(Ks);          // [16][lds], once the keys are used up
+    const size_t ks_bytes = (size_t)a.nbuf * LA_KEYS * ld * 2, os_bytes = (size_t)16 * lds * 4;
+    float* Ss = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(Ks) + (ks_bytes > os_bytes ? ks_bytes : os_bytes));
+    bf16* Ph = reinterpret_cast<bf16*>(Ss + 16 * SP);
+    bf16* Pl = Ph + 16 * PP;
+    float* corr_s = reinterpret_cast<float*>(Pl + 16 * PP);
+    float* ml_s = corr_s + 16;                          // [16][2]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int sp = blockIdx.x, hg = blockIdx.y / a.col_blocks, cb = blockIdx.y % a.col_blocks, m = blockIdx.z;
+    const int sp = blockIdx.x % CL, hg = blockIdx.x / CL, m = blockIdx.y;
+    const int hpc = 16 / CL, h_loc0 = sp * hpc, h0 = hg * 16 + h_loc0;   // heads this CTA finishes
+    const int n_fin = max(0, min(hpc, a.H - h0));
+    if constexpr (FUSE_V) {   // the value matrices are constants: on their way to L2 while the predecessor runs
+        const char* p = reinterpret_cast<const char*>(a.wuv + (size_t)h0 * a.vdim * a.Rp);
+        for (size_t i = (size_t)tid * 128; i < (size_t)n_fin * a.vdim * a.Rp * 2; i += LM_THREADS * 128)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(p + i));
+    }
     pdl_wait();
     const int slot = __ldcg(a.row_slot + m), len = __ldcg(a.row_pos + m) + 1;
     int tps, ns;
-    latent_splits(len, LA_KEYS, a.S, tps, ns);
-    if (sp >= ns) return;
-    const int k_begin = sp * tps * LA_KEYS, k_end = min(len, (sp + 1) * tps * LA_KEYS);
-    const int n_tiles = (k_end - k_begin + LA_KEYS - 1) / LA_KEYS;
+    latent_splits(len, LA_KEYS, CL, tps, ns);
+    const int k_begin = min(len, sp * tps * LA_KEYS), k_end = min(len, (sp + 1) * tps * LA_KEYS);
+    const int n_tiles = (k_end - k_begin + LA_KEYS - 1) / LA_KEYS;     // 0 for a split without keys
     const int nv = a.Dp / 8;
     const bf16* kb = static_cast<const bf16*>(a.cache) + (size_t)slot * a.max_seq * a.Dp;
-    auto fetch = [&](int tile) {
+    auto fetch = [&](int tile) {   // a tile's rows are consecutive in memory
         bf16* dst = Ks + (size_t)(tile % a.nbuf) * LA_KEYS * ld;
-        const int k0 = k_begin + tile * LA_KEYS;
-        for (int i = tid; i < LA_KEYS * nv; i += LM_THREADS) {
-            const int key = i / nv, v = i - key * nv;
-            const bool ok = k0 + key < k_end;
-            cp_async16(dst + key * ld + v * 8, kb + (size_t)(ok ? k0 + key : k_begin) * a.Dp + v * 8, ok);
-        }
+        const int k0 = k_begin + tile * LA_KEYS, n = min(LA_KEYS, k_end - k0) * nv;
+        const bf16* src = kb + (size_t)k0 * a.Dp;
+        for (int i = tid; i < LA_KEYS * nv; i += LM_THREADS)
+            cp_async16(dst + i * 8 + a.row_vecs.div(i) * 8, src + (i < n ? i : 0) * 8, i < n);
         cp_async_commit();
     };
-    {   // queries: heads hg*16 .. +15 of this row (zero rows past the last head)
-        const bf16* qb = static_cast<const bf16*>(a.q) + ((size_t)m * a.H + hg * 16) * a.Dp;
-        for (int i = tid; i < 16 * nv; i += LM_THREADS) {
-            const int h = i / nv, v = i - h * nv;
-            const bool ok = hg * 16 + h < a.H;
-            cp_async16(Qs + h * ld + v * 8, qb + (ok ? (size_t)h * a.Dp + v * 8 : 0), ok);
-        }
-    }
-    fetch(0);
     float acc[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     float m_run[2] = {NEG_BIG, NEG_BIG}, l_run[2] = {0.f, 0.f};   // heads 2*warp, 2*warp + 1
-    const int col0 = cb * NT * 64 + warp * NT * 8;
+    const int col0 = warp * NT * 8;
+    if (n_tiles > 0) {
+        // queries: heads hg*16 .. +15 of this row (zero rows past the last head)
+        const bf16* qb = static_cast<const bf16*>(a.q) + ((size_t)m * a.H + hg * 16) * a.Dp;
+        const int nq = min(16, a.H - hg * 16) * nv;
+        for (int i = tid; i < 16 * nv; i += LM_THREADS)
+            cp_async16(Qs + i * 8 + a.row_vecs.div(i) * 8, qb + (i < nq ? i : 0) * 8, i < nq);
+        fetch(0);
+    }
     const int ksteps = a.Dp / 16;
     for (int tile = 0; tile < n_tiles; ++tile) {
         const bool ahead = a.nbuf > 1 && tile + 1 < n_tiles;
@@ -137,6 +185,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
         const bf16* qp = Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
         const bf16* kp = K + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
         int ks = 0;
+#pragma unroll 4
         for (; ks + 2 <= ksteps; ks += 2) {
             uint32_t a0[4], a1[4], b[4];
             ldsm_x4(a0, qp + ks * 16);
@@ -207,22 +256,126 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
         __syncthreads();   // the tile and the weights are used up
         if (!ahead && tile + 1 < n_tiles) fetch(tile + 1);
     }
-    const size_t row = ((size_t)m * a.S + sp) * a.H + hg * 16;
+    // ---- partial sums, maxima and totals for the cluster
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
         const int col = col0 + i * 8 + 2 * t;
         if (col0 + i * 8 < a.Rp) {
-            if (hg * 16 + g < a.H) *reinterpret_cast<float2*>(a.part + (row + g) * a.Rp + col) = make_float2(acc[i][0], acc[i][1]);
-            if (hg * 16 + g + 8 < a.H)
-                *reinterpret_cast<float2*>(a.part + (row + g + 8) * a.Rp + col) = make_float2(acc[i][2], acc[i][3]);
+            *reinterpret_cast<float2*>(Os + g * lds + col) = make_float2(acc[i][0], acc[i][1]);
+            *reinterpret_cast<float2*>(Os + (g + 8) * lds + col) = make_float2(acc[i][2], acc[i][3]);
         }
     }
-    if (cb == 0 && lane == 0)
+    if (lane == 0)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int h = 2 * warp + i;
-            if (hg * 16 + h < a.H)
-                *reinterpret_cast<float2*>(a.ml + (row + h) * 2) = make_float2(m_run[i], l_run[i]);
+        for (int i = 0; i < 2; ++i) *reinterpret_cast<float2*>(ml_s + (2 * warp + i) * 2) = make_float2(m_run[i], l_run[i]);
+    cluster_arrive();
+    cluster_wait();
+    // ---- merge: 256 / hpc threads per head
+    const int tph = LM_THREADS / hpc, hl = tid / tph, c0 = tid % tph;
+    float* ol = ml_s + 32;                              // [hpc][Rp] merged sums (FUSE_V)
+    if (hl < n_fin) {
+        float w[LA_MAX_CL], mx = NEG_BIG, l = 0.f;
+        float2 p[LA_MAX_CL];
+#pragma unroll
+        for (int s = 0; s < LA_MAX_CL; ++s) {
+            p[s] = s < ns ? ld_cluster2(cluster_addr(ml_s + (h_loc0 + hl) * 2, s)) : make_float2(NEG_BIG, 0.f);
+            mx = fmaxf(mx, p[s].x);
+        }
+#pragma unroll
+        for (int s = 0; s < LA_MAX_CL; ++s) {
+            w[s] = __expf(p[s].x - mx);
+            l = fmaf(w[s], p[s].y, l);
+        }
+        const float inv = 1.0f / l;
+        for (int c = c0; c < a.Rp; c += tph) {
+            float o = 0.f;
+#pragma unroll
+            for (int s = 0; s < LA_MAX_CL; ++s)
+                if (s < ns) o = fmaf(w[s], ld_cluster(cluster_addr(Os + (h_loc0 + hl) * lds + c, s)), o);
+            if constexpr (FUSE_V) ol[hl * a.Rp + c] = o * inv;
+            else a.out[((size_t)m * a.H + h0 + hl) * a.Rp + c] = f2bf(o * inv);
+        }
+    }
+    __syncwarp();
+    cluster_arrive();
+    if constexpr (FUSE_V) {
+        __syncthreads();
+        // rows (head, d) of the value matrices, four at a time per warp
+        const int n_rows = n_fin * a.vdim, nvr = a.Rp / 8;
+        const bf16* W = a.wuv + (size_t)h0 * a.vdim * a.Rp;
+        for (int r0 = warp * 4; r0 < n_rows; r0 += LM_WARPS * 4) {
+            float s[4] = {0.f, 0.f, 0.f, 0.f};
+            for (int v = lane; v < nvr; v += 32) {
+                uint4 w[4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) w[u] = ldg_stream(W + (size_t)min(r0 + u, n_rows - 1) * a.Rp + v * 8);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const float* o = ol + (min(r0 + u, n_rows - 1) / a.vdim) * a.Rp + v * 8;
+                    float f[8];
+                    unpack8(w[u], f);
+                    const float4 x = *reinterpret_cast<const float4*>(o), y = *reinterpret_cast<const float4*>(o + 4);
+                    s[u] = fmaf(f[0], x.x, fmaf(f[1], x.y, fmaf(f[2], x.z, fmaf(f[3], x.w, s[u]))));
+                    s[u] = fmaf(f[4], y.x, fmaf(f[5], y.y, fmaf(f[6], y.z, fmaf(f[7], y.w, s[u]))));
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < 4; ++u) s[u] = warp_sum(s[u]);
+            if (lane < 4 && r0 + lane < n_rows) {
+                const size_t c = (size_t)h0 * a.vdim + r0 + lane;
+                a.out[(size_t)m * a.ldo + c] = f2bf(pick<4>(s, lane) * bf2f(a.gate[(size_t)m * a.ldgate + c]));
+            }
+        }
+    }
+    cluster_wait();   // a peer may still have been reading this CTA's sums
+}
+
+// Many rows: out[m][h*vdim + d] = gate * sum_k W_uv[h][d][k] o[m][h][k] as one small product per head.  A warp owns 16
+// value rows (the M side) and 32 activation rows (the N side); k is taken in the lanes' own order as in k_lm_stream.
+struct LatentValueArgs {
+    const bf16* wuv;       // (H, vdim, Rp)
+    const bf16* o;         // (M, H, Rp)
+    const bf16* gate; int ldgate;
+    bf16* out; int ldo;
+    int H, Rp, vdim, M;
+};
+
+static __global__ void __launch_bounds__(128) k_latent_value(LatentValueArgs a) {
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.x, d0 = (blockIdx.y * 4 + warp) * 16, m0 = blockIdx.z * 32;
+    const int nkb = a.Rp / 32;                       // Rp is a multiple of 16: a half block may be left
+    const bf16* w0 = a.wuv + ((size_t)h * a.vdim + min(d0 + g, a.vdim - 1)) * a.Rp + t * 8;
+    const bf16* w1 = a.wuv + ((size_t)h * a.vdim + min(d0 + g + 8, a.vdim - 1)) * a.Rp + t * 8;
+    const bf16* o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = a.o + ((size_t)min(m0 + j * 8 + g, a.M - 1) * a.H + h) * a.Rp + t * 8;
+    float acc[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    pdl_wait();
+    if (d0 >= a.vdim) return;
+    const int blocks = (a.Rp + 31) / 32;
+    for (int b = 0; b < blocks; ++b) {
+        const bool in = b < nkb || t < 2;            // lanes 2, 3 of a half block hold zeros
+        const uint4 x0 = in ? ldg_stream(w0 + b * 32) : make_uint4(0, 0, 0, 0), x1 = in ? ldg_stream(w1 + b * 32) : make_uint4(0, 0, 0, 0);
+        const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const uint4 y = in ? __ldcg(reinterpret_cast<const uint4*>(o[j] + b * 32)) : make_uint4(0, 0, 0, 0);
+            mma_bf16(acc[j], a0, y.x, y.y);
+            mma_bf16(acc[j], a1, y.z, y.w);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int d = d0 + g + (c >> 1) * 8, m = m0 + j * 8 + 2 * t + (c & 1);
+            if (d < a.vdim && m < a.M) {
+                const size_t col = (size_t)h * a.vdim + d;
+                a.out[(size_t)m * a.ldo + col] = f2bf(acc[j][c] * bf2f(a.gate[(size_t)m * a.ldgate + col]));
+            }
         }
 }
 

@@ -51,6 +51,7 @@ struct LatentPrefillArgs {
     bf16* out; int ldo;
     int H, dimp, rotp, vdim, vdp, Rp, Dp, max_seq;
     float scale;
+    FastDiv key_vecs;        // 16-byte pieces of a key and its value
 };
 
 static inline size_t latent_prefill_smem(int qk, int v) { return (size_t)2 * LP_TILE * (qk + 8 + v + 8) * 2; }
@@ -75,7 +76,7 @@ static __global__ void __launch_bounds__(128) k_latent_prefill(LatentPrefillArgs
         bf16* kd = Ks + (size_t)buf * LP_TILE * ldk;
         bf16* vd = Vs + (size_t)buf * LP_TILE * ldv;
         for (int i = tid; i < LP_TILE * n_all; i += 128) {
-            const int key = i / n_all, v = i - key * n_all;
+            const int key = a.key_vecs.div(i), v = i - key * n_all;
             const bool ok = k0 + key < n_keys;
             const size_t p = ok ? k0 + key : 0;
             if (v < n_kv) cp_async16(kd + key * ldk + v * 8, kx + p * a.ldx + v * 8, ok);

@@ -1,11 +1,11 @@
 // libvuib200_lm: C ABI over the token-model kernels (see include/vuib200_lm.h).  The host side validates, lays out the
 // caller's workspace and enqueues kernels on the caller's stream; it never allocates device memory.
 //
-// A layer is five launches for up to LM_GEMV_ROWS rows
-//   [norms + every projection of x] [queries, cache append] [attention splits] [merge, value matrix, gate] [output + MLP
-//   down, residual]
-// and seven for more: row norms, tcgen05 GEMM, latent rows, tcgen05 GEMM, attention, merge, tcgen05 GEMM.  A prefill
-// of many rows expands keys and values instead (latent_attn.cuh).
+// A layer is four launches for up to LM_FEW_ROWS rows
+//   [norms + every projection of x] [queries, cache append] [attention, value matrix, gate] [output + MLP down, residual]
+// and seven for more: row norms, tcgen05 GEMM, latent rows, tcgen05 GEMM, attention, value matrix, tcgen05 GEMM.  A
+// prefill of many rows expands keys and values instead (latent_prefill.cuh).  32-bit models: fp32 products, and the
+// attention's splits merge in a launch of their own.
 #include "../../include/vuib200_lm.h"
 
 #include <cstdarg>
@@ -26,14 +26,15 @@ using namespace vuib;
 
 namespace {
 
-constexpr int LM_GEMV_ROWS = 4;        // rows up to which the weight-streaming GEMV runs
-constexpr int LA_ROW_BLOCK = 512;      // rows of one absorbed-attention launch (bounds the split scratch)
-constexpr int LA_CTAS = 2 * 148;       // CTAs the key splits of a few rows are cut to
+constexpr int LM_FEW_ROWS = 8;         // rows up to which the weight-streaming products run (fp32: 4)
+constexpr int LM_FEW_ROWS_F32 = 4;
+constexpr int LA_ROW_BLOCK = 512;      // rows of one fp32 attention launch (bounds the split scratch)
+constexpr int LA_CTAS = 2 * 148;       // CTAs of one wave: what rows of weights and splits of keys are cut to
 constexpr int LM_EXPAND_MIN = 64;      // rows of a call from which a prefill expands keys and values
 constexpr size_t LM_MAX_SMEM = 227 * 1024;
 
 struct LmLayout {
-    size_t flag, ctl, row_slot, row_pos, segs, xsegs, tiles, x, xn, dq, cq, dkv, gate, q, ay, part, ml;
+    size_t flag, ctl, row_slot, row_pos, segs, xsegs, tiles, x, xn, dq, cq, dkv, gate, q, ay, part, ml, olat;
     size_t tc_partial, tc_counters, xkv, xc;
     size_t draw_ctr, rep_counts, rep_hist, rep_head, rep_filled;
     size_t total;
@@ -61,6 +62,7 @@ struct VuibLm {
     LmLayout lay;
     bool have_w, have_cache, have_ws;
     int R;                 // rows of scratch
+    int few_rows;          // rows up to which the streaming products run for this model's sizes
     int num_sms;
     unsigned spin_limit;
     int expand_min;
@@ -141,7 +143,7 @@ void make_layout(VuibLm* e) {
     const size_t R = e->R, es = c.dtype == VUIB_LM_BF16 ? 2 : 4;
     size_t off = 0;
     auto take = [&](size_t bytes) { size_t o = off; off = align_up(off + bytes); return o; };
-    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0;
+    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0, olat = 0;
     size_t part = 0, ml = 0;
     for (size_t i = 0; i < e->layer.size(); ++i) {
         const VuibLmLayer& l = e->layer[i];
@@ -158,7 +160,8 @@ void make_layout(VuibLm* e) {
             mx(xc, d.k_kv);
         }
         mx(ay, d.k_out);
-        for (int m = 1; m <= LA_ROW_BLOCK && m <= (int)R; ++m) {
+        mx(olat, l.heads * d.rp);
+        for (int m = 1; c.dtype == VUIB_LM_F32 && m <= LA_ROW_BLOCK && m <= (int)R; ++m) {
             const size_t rows = (size_t)m * attn_splits(e, (int)i, m) * l.heads;
             if (rows * d.rp > part) part = rows * d.rp;
             if (rows * 2 > ml) ml = rows * 2;
@@ -188,6 +191,7 @@ void make_layout(VuibLm* e) {
     L.ay = take(R * ay * es);
     L.part = take(part * 4);
     L.ml = take(ml * 4);
+    L.olat = take(c.dtype == VUIB_LM_BF16 ? R * olat * 2 : 0);
     L.tc_partial = take(c.dtype == VUIB_LM_BF16 ? tc_partial_bytes(R + L.x_rows) : 0);
     L.tc_counters = take(2 * TC_COUNTERS * 4);
     L.xkv = take((size_t)L.x_rows * xkv * es);
@@ -216,34 +220,94 @@ cudaError_t allow_smem(const void* kern, size_t bytes) {
 }
 
 template <class... KArgs, class... Args>
-int32_t run(VuibLm* e, void (*kern)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t s, Args... args) {
+int32_t run_cl(VuibLm* e, void (*kern)(KArgs...), dim3 grid, int cluster, int threads, size_t smem, cudaStream_t s, Args... args) {
     CK(allow_smem(reinterpret_cast<const void*>(kern), smem));
-    CK(launch(kern, grid, threads, smem, s, args...));
+    CK(launch_cl(kern, grid, cluster, threads, smem, s, args...));
     e->launches++;
     return VUIB_OK;
+}
+
+template <class... KArgs, class... Args>
+int32_t run(VuibLm* e, void (*kern)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t s, Args... args) {
+    return run_cl(e, kern, grid, 1, threads, smem, s, args...);
 }
 
 // ---------------------------------------------------------------------------
 // Matrix products
 // ---------------------------------------------------------------------------
-template <class T, int RT, class Stage, class Epi>
+constexpr size_t LS_MAX_SMEM = 200 * 1024;
+
+// CTAs of a cluster along K for a product whose rows alone do not fill the SMs.
+int stream_ck(int n_groups, int K, bool k_parts) {
+    int ck = 1;
+    while (k_parts && ck < 4 && n_groups * ck * 2 <= LA_CTAS && K % (64 * ck) == 0 && K / (2 * ck) >= 256) ck *= 2;
+    return ck;
+}
+
+size_t stream_smem(int tiles, int rt, int K, int ck) { return (size_t)tiles * rt * (K / ck + LS_PAD) * 2; }
+
+template <int RT, class Stage, class Epi>
+int32_t stream_rt(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int K, int M, int n_rows, cudaStream_t s) {
+    StreamArgs a;
+    a.W = static_cast<const bf16*>(W);
+    a.K = K;
+    a.M = M;
+    a.n_groups = (n_rows + 15) / 16;
+    a.ck = stream_ck(a.n_groups, K, Stage::K_PARTS);
+    // warps along K: as many as the one wave of CTAs has to spare, two 32-k blocks each at least
+    a.kw = 1;
+    const int blocks = K / a.ck / 32;
+    while (a.kw < LM_WARPS && a.n_groups * a.ck * a.kw * 2 <= LA_CTAS * LM_WARPS && a.kw * 4 <= blocks) a.kw *= 2;
+    const int gpc = LM_WARPS / a.kw, need = (a.n_groups + gpc - 1) / gpc, most = LA_CTAS / a.ck;
+    const int sets = (need + most - 1) / most, ctas = (need + sets - 1) / sets;
+    return run_cl(e, k_lm_stream<RT, Stage, Epi>, dim3(ctas * a.ck + (Stage::HAS_EXTRA ? 1 : 0)), a.ck, LM_THREADS,
+                  stream_smem(Stage::TILES, RT, K, a.ck), s, st, ep, a);
+}
+
+template <int RT, class Stage, class Epi>
 int32_t gemv_rt(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int K, int M, int n_pairs, cudaStream_t s) {
-    const int nv = K / Store<T>::VEC;
+    const int nv = K / Store<float>::VEC;
     int wk = 1;   // warps along K: enough CTAs for every SM, at least one vector per lane
     while (wk < LM_WARPS && (n_pairs + LM_WARPS / wk - 1) / (LM_WARPS / wk) < LA_CTAS && 32 * wk < nv) wk *= 2;
     const int per = LM_WARPS / wk, grid = (n_pairs + per - 1) / per + (Stage::HAS_EXTRA ? 1 : 0);
-    return run(e, k_lm_gemv<T, RT, Stage, Epi>, dim3(grid), LM_THREADS, Stage::smem(RT, K), s, st, ep,
-               static_cast<const T*>(W), K, M, n_pairs, wk);
+    return run(e, k_lm_gemv<float, RT, Stage, Epi>, dim3(grid), LM_THREADS, Stage::smem(RT, K), s, st, ep,
+               static_cast<const float*>(W), K, M, n_pairs, wk);
 }
 
+// n_rows weight rows times up to few_rows activation rows.
 template <class T, class Stage, class Epi>
-int32_t gemv(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int K, int M, int n_rows, cudaStream_t s) {
-    const int n_pairs = (n_rows + 1) / 2;
-    const size_t most = LM_MAX_SMEM - 8 * 1024;
-    if (M > 2 && Stage::smem(4, K) <= most) return gemv_rt<T, 4>(e, st, ep, W, K, M, n_pairs, s);
-    if (M > 1 && Stage::smem(2, K) <= most) return gemv_rt<T, 2>(e, st, ep, W, K, M, n_pairs, s);
-    if (Stage::smem(1, K) <= most) return gemv_rt<T, 1>(e, st, ep, W, K, M, n_pairs, s);
-    return fail(e, VUIB_ERR_SHAPE, "a row of %d elements does not fit shared memory", K);
+int32_t few(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int K, int M, int n_rows, cudaStream_t s) {
+    if constexpr (std::is_same<T, bf16>::value) {
+        if (M <= 1) return stream_rt<1>(e, st, ep, W, K, M, n_rows, s);
+        if (M <= 2) return stream_rt<2>(e, st, ep, W, K, M, n_rows, s);
+        if (M <= 4) return stream_rt<4>(e, st, ep, W, K, M, n_rows, s);
+        return stream_rt<8>(e, st, ep, W, K, M, n_rows, s);
+    } else {
+        const int n_pairs = (n_rows + 1) / 2;
+        if (M > 2 && Stage::smem(4, K) <= LS_MAX_SMEM) return gemv_rt<4>(e, st, ep, W, K, M, n_pairs, s);
+        if (M > 1 && Stage::smem(2, K) <= LS_MAX_SMEM) return gemv_rt<2>(e, st, ep, W, K, M, n_pairs, s);
+        return gemv_rt<1>(e, st, ep, W, K, M, n_pairs, s);
+    }
+}
+
+// Rows up to which `few` fits shared memory in every product of the model (0: not even one).
+int few_rows_of(const VuibLm* e) {
+    const VuibLmConfig& c = e->cfg;
+    const bool b16 = c.dtype == VUIB_LM_BF16;
+    for (int rt = b16 ? LM_FEW_ROWS : LM_FEW_ROWS_F32; rt >= 1; rt /= 2) {
+        bool ok = true;
+        for (const VuibLmDims& d : e->dims) {
+            if (b16) {
+                ok = ok && stream_smem(2, rt, d.k_in, 1) <= LS_MAX_SMEM && stream_smem(1, rt, d.k_q, 1) <= LS_MAX_SMEM &&
+                     stream_smem(1, rt, d.k_out, stream_ck(up(c.width, 16) / 16, d.k_out, true)) <= LS_MAX_SMEM;
+            } else {   // one row at a time will do
+                ok = ok && StageLayerNorm2<float>::smem(1, d.k_in) <= LS_MAX_SMEM && StageRowsT<float>::smem(1, d.k_out) <= LS_MAX_SMEM &&
+                     StageRowsT<float>::smem(1, d.k_q) <= LS_MAX_SMEM;
+            }
+        }
+        if (ok) return rt;
+    }
+    return 0;
 }
 
 // Rows [row_off, row_off + n_rows) of W (n_rows a multiple of 128) times M rows of X; weight rows >= n_split (counted
@@ -254,7 +318,7 @@ int32_t gemm(VuibLm* e, const CUtensorMap& map, const void* W, const T* X, int l
     if constexpr (std::is_same<T, bf16>::value) {
         const TcCtx cx{wsp<float>(e, e->lay.tc_partial), wsp<int32_t>(e, e->lay.tc_counters), wsp<int32_t>(e, e->lay.flag),
                        nullptr, &e->num_sms, e->spin_limit, &e->launches};
-        CK(tc_gemm_launch(cx, map, map, X, ldx, M, K, n_rows, 0, TcPair<Epi>{ep}, s,
+        CK(tc_gemm_launch(cx, map, map, X, ldx, M, K, n_rows, 0, typename TcForm<Epi>::type{ep}, s,
                           n_split < n_rows ? n_split / TC_TILE_N : 1 << 30, n_split < n_rows ? x_off : 0));
         return VUIB_OK;
     } else {
@@ -266,70 +330,109 @@ int32_t gemm(VuibLm* e, const CUtensorMap& map, const void* W, const T* X, int l
 // ---------------------------------------------------------------------------
 // Attention
 // ---------------------------------------------------------------------------
-template <class T>
-int32_t absorbed_attention(VuibLm* e, int li, int M, cudaStream_t s) {
-    const VuibLmConfig& c = e->cfg;
+LatentAttnArgs attn_args(VuibLm* e, int li) {
     const VuibLmLayer& l = e->layer[li];
     const VuibLmDims& d = e->dims[li];
     const LmLayout& L = e->lay;
-    constexpr bool B16 = std::is_same<T, bf16>::value;
+    LatentAttnArgs a;
+    memset(&a, 0, sizeof(a));
+    a.q = e->ws + L.q;
+    a.cache = e->cache[li];
+    a.row_slot = wsp<int32_t>(e, L.row_slot);
+    a.row_pos = wsp<int32_t>(e, L.row_pos);
+    a.H = l.heads;
+    a.Rp = d.rp;
+    a.Dp = d.dp;
+    a.max_seq = e->cfg.max_seq;
+    a.scale = l.scale;
+    a.row_vecs = FastDiv(d.dp / 8);
+    return a;
+}
+
+template <bool FUSE_V>
+int32_t latent_attn_nt(VuibLm* e, const LatentAttnArgs& a, int CL, int M, cudaStream_t s) {
+    const dim3 grid(CL * ((a.H + 15) / 16), M);
+    const size_t sm = latent_attn_smem(a.Dp, a.Rp, a.nbuf, FUSE_V ? 16 / CL : 0);
+    if (a.Rp <= 128) return run_cl(e, k_latent_attn<2, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
+    if (a.Rp <= 256) return run_cl(e, k_latent_attn<4, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
+    if (a.Rp <= 512) return run_cl(e, k_latent_attn<8, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
+    return run_cl(e, k_latent_attn<16, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
+}
+
+int32_t absorbed_attention_bf16(VuibLm* e, int li, int M, cudaStream_t s) {
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    const LmLayout& L = e->lay;
+    LatentAttnArgs a = attn_args(e, li);
+    // splits of a row's keys: one wave of CTAs, no more than the cache has tiles
+    const int units = M * ((l.heads + 15) / 16);
+    int CL = 1;
+    while (CL < LA_MAX_CL && units * CL * 2 <= LA_CTAS && CL * LA_KEYS < e->cfg.max_seq) CL *= 2;
+    a.nbuf = latent_attn_smem(d.dp, d.rp, 2, 16) <= LM_MAX_SMEM ? 2 : 1;
+    a.wuv = static_cast<const bf16*>(e->w[li].w_uv);
+    a.gate = wsp<bf16>(e, L.gate);
+    a.ldgate = L.ld_gate;
+    a.vdim = l.vdim;
+    a.ldo = L.ld_ay;
+    if (M <= LM_FEW_ROWS) {
+        a.out = wsp<bf16>(e, L.ay);
+        return latent_attn_nt<true>(e, a, CL, M, s);
+    }
+    a.out = wsp<bf16>(e, L.olat);
+    RC(latent_attn_nt<false>(e, a, CL, M, s));
+    const LatentValueArgs v{a.wuv, wsp<bf16>(e, L.olat), a.gate, L.ld_gate, wsp<bf16>(e, L.ay), L.ld_ay, l.heads, d.rp, l.vdim, M};
+    return run(e, k_latent_value, dim3(l.heads, (l.vdim + 63) / 64, (M + 31) / 32), 128, 0, s, v);
+}
+
+int32_t absorbed_attention_f32(VuibLm* e, int li, int M, cudaStream_t s) {
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    const LmLayout& L = e->lay;
     for (int m0 = 0; m0 < M; m0 += LA_ROW_BLOCK) {
         const int m = M - m0 < LA_ROW_BLOCK ? M - m0 : LA_ROW_BLOCK;
-        LatentAttnArgs a;
-        a.q = wsp<T>(e, L.q) + (size_t)m0 * l.heads * d.dp;
-        a.cache = e->cache[li];
-        a.row_slot = wsp<int32_t>(e, L.row_slot) + m0;
-        a.row_pos = wsp<int32_t>(e, L.row_pos) + m0;
+        LatentAttnArgs a = attn_args(e, li);
+        a.q = wsp<float>(e, L.q) + (size_t)m0 * l.heads * d.dp;
+        a.row_slot += m0;
+        a.row_pos += m0;
         a.part = wsp<float>(e, L.part);
         a.ml = wsp<float>(e, L.ml);
-        a.H = l.heads;
-        a.Rp = d.rp;
-        a.Dp = d.dp;
-        a.max_seq = c.max_seq;
         a.S = attn_splits(e, li, m);
-        a.scale = l.scale;
-        const int hg = (l.heads + 15) / 16;
-        if constexpr (B16) {
-            a.nbuf = latent_attn_smem(d.dp, 2) <= LM_MAX_SMEM ? 2 : 1;
-            const size_t sm = latent_attn_smem(d.dp, a.nbuf);
-            const int nt = d.rp <= 128 ? 2 : d.rp <= 256 ? 4 : 8;
-            a.col_blocks = (d.rp + nt * 64 - 1) / (nt * 64);
-            const dim3 grid(a.S, hg * a.col_blocks, m);
-            if (nt == 2) RC(run(e, k_latent_attn<2>, grid, LM_THREADS, sm, s, a));
-            else if (nt == 4) RC(run(e, k_latent_attn<4>, grid, LM_THREADS, sm, s, a));
-            else RC(run(e, k_latent_attn<8>, grid, LM_THREADS, sm, s, a));
-        } else {
-            a.nbuf = 1;
-            const int nc = d.rp <= 128 ? 8 : 32;
-            a.col_blocks = (d.rp + nc * 16 - 1) / (nc * 16);
-            const dim3 grid(a.S, hg * a.col_blocks, m);
-            const size_t sm = latent_attn_f32_smem(d.dp);
-            if (nc == 8) RC(run(e, k_latent_attn_f32<8>, grid, LM_THREADS, sm, s, a));
-            else RC(run(e, k_latent_attn_f32<32>, grid, LM_THREADS, sm, s, a));
-        }
+        a.nbuf = 1;
+        const int nc = d.rp <= 128 ? 8 : 32;
+        a.col_blocks = (d.rp + nc * 16 - 1) / (nc * 16);
+        const dim3 grid(a.S, (l.heads + 15) / 16 * a.col_blocks, m);
+        const size_t sm = latent_attn_f32_smem(d.dp);
+        if (nc == 8) RC(run(e, k_latent_attn_f32<8>, grid, LM_THREADS, sm, s, a));
+        else RC(run(e, k_latent_attn_f32<32>, grid, LM_THREADS, sm, s, a));
         LatentOutArgs o;
         o.part = a.part;
         o.ml = a.ml;
         o.row_pos = a.row_pos;
         o.wuv = e->w[li].w_uv;
-        o.gate = wsp<T>(e, L.gate) + (size_t)m0 * L.ld_gate;
+        o.gate = wsp<float>(e, L.gate) + (size_t)m0 * L.ld_gate;
         o.ldgate = L.ld_gate;
-        o.out = wsp<T>(e, L.ay) + (size_t)m0 * L.ld_ay;
+        o.out = wsp<float>(e, L.ay) + (size_t)m0 * L.ld_ay;
         o.ldo = L.ld_ay;
         o.H = l.heads;
         o.Rp = d.rp;
         o.vdim = l.vdim;
         o.S = a.S;
-        o.keys = B16 ? LA_KEYS : LA_KEYS_F32;
+        o.keys = LA_KEYS_F32;
         o.M = m;
         const int rt = m == 1 ? 1 : 4, rows = (m + rt - 1) / rt;
         int vs = (148 + l.heads * rows - 1) / (l.heads * rows);   // slices of the value dimensions, >= 8 each
         if (vs > (l.vdim + 7) / 8) vs = (l.vdim + 7) / 8;
-        const dim3 grid(l.heads, rows, vs);
-        if (rt == 1) RC(run(e, k_latent_out<T, 1>, grid, LM_THREADS, (size_t)d.rp * 4, s, o));
-        else RC(run(e, k_latent_out<T, 4>, grid, LM_THREADS, (size_t)4 * d.rp * 4, s, o));
+        const dim3 og(l.heads, rows, vs);
+        if (rt == 1) RC(run(e, k_latent_out<float, 1>, og, LM_THREADS, (size_t)d.rp * 4, s, o));
+        else RC(run(e, k_latent_out<float, 4>, og, LM_THREADS, (size_t)4 * d.rp * 4, s, o));
     }
     return VUIB_OK;
+}
+
+template <class T>
+int32_t absorbed_attention(VuibLm* e, int li, int M, cudaStream_t s) {
+    if constexpr (std::is_same<T, bf16>::value) return absorbed_attention_bf16(e, li, M, s);
+    else return absorbed_attention_f32(e, li, M, s);
 }
 
 struct ExpandGroup {   // sequences of a prefill whose keys are expanded together
@@ -367,6 +470,7 @@ int32_t expanded_attention(VuibLm* e, int li, const ExpandGroup& g, cudaStream_t
     a.Dp = d.dp;
     a.max_seq = c.max_seq;
     a.scale = l.scale;
+    a.key_vecs = FastDiv((d.dimp + d.rotp + d.vdp) / 8);
     const int qk = d.dimp + d.rotp;
     const size_t sm = latent_prefill_smem(qk, d.vdp);
     const dim3 grid(g.n_tiles, l.heads);
@@ -388,13 +492,13 @@ int32_t run_layers(VuibLm* e, int M, const std::vector<ExpandGroup>* expand, cud
     const VuibLmConfig& c = e->cfg;
     const LmLayout& L = e->lay;
     float* x = wsp<float>(e, L.x);
-    const bool few = M <= LM_GEMV_ROWS;
+    const bool stream = M <= e->few_rows;
     for (int li = 0; li < c.n_layers; ++li) {
         const VuibLmLayer& l = e->layer[li];
         const VuibLmDims& d = e->dims[li];
         const VuibLmLayerWeights& w = e->w[li];
         const LmMaps& mp = e->maps[li];
-        const bool ex = expand && d.x_ok && !few;
+        const bool ex = expand && d.x_ok && !stream;
         const LayerNormW n1{w.norm1_w, w.norm1_b}, n2{w.norm2_w, w.norm2_b};
         const float2* trig = reinterpret_cast<const float2*>(w.trig);
         T* ay = wsp<T>(e, L.ay);
@@ -421,14 +525,14 @@ int32_t run_layers(VuibLm* e, int M, const std::vector<ExpandGroup>* expand, cud
         const EpRotatedQ<T> eq{wsp<T>(e, L.q), l.heads * head_rows, head_rows, head_rows - d.rotp, l.rot_dims, trig,
                                wsp<int32_t>(e, L.row_pos)};
         const EpAddResidual er{x, L.ldx, c.width};
-        if (few) {
+        if (stream) {
             const StageLayerNorm2<T> sn{x, L.ldx, c.width, c.norm_eps, n1, n2, d.n_mlp, nullptr};
-            RC(gemv<T>(e, sn, ei, w.w_in, d.k_in, M, d.n_in, s));
+            RC(few<T>(e, sn, ei, w.w_in, d.k_in, M, d.n_in, s));
             const StageLatentQ<T> sq{wsp<float>(e, L.dq), L.ld_dq, l.q_rank, c.norm_eps, w.q_norm, lat};
-            RC(gemv<T>(e, sq, eq, w.w_q, d.k_q, M, l.heads * d.dp, s));
+            RC(few<T>(e, sq, eq, w.w_q, d.k_q, M, l.heads * d.dp, s));
             RC(absorbed_attention<T>(e, li, M, s));
             const StageRowsT<T> sr{ay, L.ld_ay};
-            RC(gemv<T>(e, sr, er, w.w_out, d.k_out, M, c.width, s));
+            RC(few<T>(e, sr, er, w.w_out, d.k_out, M, c.width, s));
         } else {
             T* xn = wsp<T>(e, L.xn);
             T* xn2 = xn + (size_t)e->R * L.ldx;
@@ -465,7 +569,7 @@ int32_t run_head(VuibLm* e, int M, const int32_t* rows, const int32_t* row_slot,
            LayerNormW{e->head.final_w, e->head.final_b}, xn, LayerNormW{nullptr, nullptr}, static_cast<T*>(nullptr), L.ldx, rows,
            row_slot, seq_inc, seq_lens));
     const EpLogitsF32 el{logits, c.vocab};
-    if (M <= LM_GEMV_ROWS) return gemv<T>(e, StageRowsT<T>{xn, L.ldx}, el, e->head.head, L.ldx, M, c.vocab, s);
+    if (M <= e->few_rows) return few<T>(e, StageRowsT<T>{xn, L.ldx}, el, e->head.head, L.ldx, M, c.vocab, s);
     return gemm<T>(e, e->map_head, e->head.head, xn, L.ldx, L.ldx, M, up(c.vocab, 128), el, s);
 }
 
@@ -544,7 +648,8 @@ extern "C" int32_t vuib_lm_create(const VuibLmConfig* cfg, const VuibLmLayer* la
             return VUIB_ERR_SHAPE;
         if (l.mlp != VUIB_LM_MLP_NONE && l.ff < 1) return VUIB_ERR_SHAPE;
         const VuibLmDims d = layer_dims(c, l);
-        if (c.dtype == VUIB_LM_BF16 ? latent_attn_smem(d.dp, 1) > LM_MAX_SMEM : latent_attn_f32_smem(d.dp) > LM_MAX_SMEM)
+        if (c.dtype == VUIB_LM_BF16 ? d.rp > 1024 || latent_attn_smem(d.dp, d.rp, 1, 16) > LM_MAX_SMEM
+                                    : latent_attn_f32_smem(d.dp) > LM_MAX_SMEM)
             return VUIB_ERR_SHAPE;
     }
     VuibLm* e = new (std::nothrow) VuibLm();
@@ -558,6 +663,7 @@ extern "C" int32_t vuib_lm_create(const VuibLmConfig* cfg, const VuibLmLayer* la
     e->R = c.max_rows > c.max_prefill_rows ? c.max_rows : c.max_prefill_rows;
     e->spin_limit = TC_SPIN_LIMIT;
     e->expand_min = LM_EXPAND_MIN;
+    e->few_rows = few_rows_of(e);
     make_layout(e);
     *out = e;
     return VUIB_OK;
@@ -655,7 +761,7 @@ extern "C" int32_t vuib_lm_prefill(VuibLm* e, int32_t n_segs, const int32_t* slo
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     CK(cudaMemcpyAsync(e->ws + e->lay.segs, segs.data(), segs.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
     std::vector<ExpandGroup> groups;
-    if (e->lay.x_rows && rows >= e->expand_min && rows > LM_GEMV_ROWS) {
+    if (e->lay.x_rows && rows >= e->expand_min && rows > e->few_rows) {
         // sequences are expanded together while their keys fit the scratch (one sequence always does); tiles with the
         // most keys first
         std::vector<int4> xsegs, tiles;

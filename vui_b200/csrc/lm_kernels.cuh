@@ -294,29 +294,45 @@ struct EpRotatedQ {
     T* q; int N, head_rows, n0, rot_dims;
     const float2* trig;
     const int32_t* row_pos;
-    __device__ __forceinline__ void store(int m, int n, float v0, float v1) const {
-        if (n >= N) return;
-        const int j = n % head_rows - n0;
+    __device__ __forceinline__ void put(int m, int n, int j, float v0, float v1, const float2* tr) const {
         if (j >= 0 && j < rot_dims) {
-            const float2 o = rotate_pair(v0, v1, __ldg(trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) + (j >> 1)));
+            const float2 o = rotate_pair(v0, v1, tr[j >> 1]);
             v0 = o.x;
             v1 = o.y;
         }
         Store<T>::put2(q + (size_t)m * N + n, v0, v1);
     }
+    __device__ __forceinline__ void store(int m, int n, float v0, float v1) const {
+        if (n >= N) return;
+        const int j = n % head_rows - n0;
+        put(m, n, j, v0, v1, j >= 0 && j < rot_dims ? trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) : nullptr);
+    }
+    // tcgen05 form: the rows' (cos, sin) are fetched while the MMAs run, TC_EPI_BYTES_PER_M of them per row
+    static constexpr int STAGE_DIMS = TC_EPI_BYTES_PER_M / 4;
+    __device__ __forceinline__ void stage(unsigned char* es, int m_off, int M, int tid) const {
+        if (rot_dims > STAGE_DIMS) return;
+        const int half = rot_dims / 2;
+        float2* dst = reinterpret_cast<float2*>(es);
+        for (int m = tid; m < M; m += TC_THREADS) {
+            const float2* src = trig + (size_t)__ldcg(row_pos + m_off + m) * half;
+            for (int i = 0; i < half; ++i) dst[m * half + i] = __ldg(src + i);
+        }
+    }
+    __host__ __device__ size_t stage_bytes_per_row() const { return rot_dims <= STAGE_DIMS ? (size_t)rot_dims * 4 : 0; }
+    __device__ __forceinline__ void store_staged(int m_off, int m, int n, float v0, float v1, const unsigned char* es) const {
+        if (rot_dims > STAGE_DIMS) return store(m_off + m, n, v0, v1);
+        if (n < N) put(m_off + m, n, n % head_rows - n0, v0, v1, reinterpret_cast<const float2*>(es) + m * (rot_dims / 2));
+    }
 };
 
-// x += W a in 32 bits.
+// x += W a in 32 bits.  Every element is added to once per launch, so the reductions have no order to depend on; they
+// return nothing, so no thread waits for the old value.
 struct EpAddResidual {
     float* x; int ldx, N;
     __device__ __forceinline__ void store(int m, int n, float v0, float v1) const {
         float* p = x + (size_t)m * ldx + n;
-        if (n + 1 < N) {
-            float2 o = __ldcg(reinterpret_cast<const float2*>(p));
-            *reinterpret_cast<float2*>(p) = make_float2(o.x + v0, o.y + v1);
-        } else if (n < N) {
-            *p = __ldcg(p) + v0;
-        }
+        if (n + 1 < N) asm volatile("red.global.add.v2.f32 [%0], {%1, %2};" ::"l"(p), "f"(v0), "f"(v1) : "memory");
+        else if (n < N) atomicAdd(p, v0);
     }
 };
 
@@ -360,11 +376,42 @@ struct TcPair {
     }
 };
 
+// The same for a functor that fetches something per activation row while the MMAs run.
+template <class F>
+struct TcPairStaged {
+    F f;
+    int m_off = 0;
+    static constexpr bool PAIRED = false;
+    static constexpr bool STAGED = true;
+    __host__ __device__ TcPairStaged shifted(int m) const { return TcPairStaged{f, m_off + m}; }
+    size_t stage_bytes_per_row() const { return f.stage_bytes_per_row(); }
+    __device__ __forceinline__ void stage(unsigned char* es, int, int M, int tid) const { f.stage(es, m_off, M, tid); }
+    __device__ __forceinline__ void apply(int n, int m0, int M, const float (&v)[8], float*, const unsigned char* es) const {
+        const bool odd = n & 1;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float give = odd ? v[j] : v[4 + j];
+            const float got = __shfl_xor_sync(0xffffffffu, give, 1);
+            const int m = m0 + j + (odd ? 4 : 0);
+            if (m < M) f.store_staged(m_off, m, n & ~1, odd ? got : v[j], odd ? v[4 + j] : got, es);
+        }
+    }
+};
+template <class F> struct TcForm { typedef TcPair<F> type; };
+template <class T> struct TcForm<EpRotatedQ<T>> { typedef TcPairStaged<EpRotatedQ<T>> type; };
+
 // ---------------------------------------------------------------------------
-// Weight-streaming GEMV for a few rows, K and N at run time.  A warp owns two adjacent weight rows; `wk` warps may
-// split K (their sums meet in shared memory in order).  Weights are requested before the dependency wait.
-// Stage functors fill X tiles [RT][K] of T in shared memory and say which tile a weight row multiplies.
+// Weight-streaming products for a few rows.  Stage functors fill X tiles [RT][K] of T in shared memory and say which
+// tile a weight row multiplies.  Weights are requested before the dependency wait.
+//
+//  k_lm_stream (bf16, up to 8 rows): a warp owns 16 weight rows (the M side of mma.sync m16n8k16) and the activation
+//  rows are its N side.  A dot product does not care about the order of k, so a lane takes 8 consecutive k of its rows
+//  with one 16-byte load and feeds them to the two MMAs of a 32-k block; the activations are read with the same
+//  permutation.  kw warps of a CTA and ck CTAs of a cluster split K; their sums meet in shared memory in order.
+//
+//  k_lm_gemv (fp32, any row count in tiles of RT): a warp owns two adjacent weight rows, wk warps may split K.
 // ---------------------------------------------------------------------------
+constexpr int LS_PAD = 32;   // elements between X rows beyond K: eight lanes of a 16-byte read hit eight bank groups
 
 // Two layer norms of the residual row (rows of W below `split` multiply the first).
 template <class T>
@@ -424,6 +471,92 @@ struct StageLayerNorm2 {
     }
     __device__ __forceinline__ void extra(int) const {}
     static constexpr bool HAS_EXTRA = false;
+
+    // k_lm_stream form: 8 / RT warps per row; (count, mean, sum of squared deviations) of the pieces are merged, so
+    // that one exchange gives mean and variance
+    static constexpr int TILES = 2;
+    static constexpr bool K_PARTS = false;
+    template <int RT>
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, int K, int M, int) const {
+        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, KEEP = 4;
+        const int r = threadIdx.x / TPR, i0 = threadIdx.x % TPR, warp = threadIdx.x >> 5;
+        const bool on = r < M;
+        const float* xr = x + (size_t)(on ? (rows ? rows[r] : r) : 0) * ldx;
+        const int nv = (width + 3) / 4;    // ldx is a multiple of 64 and the row's pad is zero
+        float4 v[KEEP];
+        float n = 0.f, mean = 0.f, m2 = 0.f;
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) {
+            const int q = i0 + i * TPR;
+            v[i] = on && q < nv ? __ldcg(reinterpret_cast<const float4*>(xr) + q) : make_float4(0.f, 0.f, 0.f, 0.f);
+            mean += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+            n += (float)max(0, min(4, width - 4 * q));
+        }
+        for (int q = i0 + KEEP * TPR; q < nv; q += TPR) {
+            const float4 u = __ldcg(reinterpret_cast<const float4*>(xr) + q);
+            mean += (u.x + u.y) + (u.z + u.w);
+            n += (float)min(4, width - 4 * q);
+        }
+        mean = n > 0.f ? mean / n : 0.f;
+        auto dev = [&](const float4& u, int q) {
+            const float a = u.x - mean, b = u.y - mean, c = u.z - mean, d = u.w - mean;
+            const int left = width - 4 * q;
+            if (left > 0) m2 = fmaf(a, a, m2);
+            if (left > 1) m2 = fmaf(b, b, m2);
+            if (left > 2) m2 = fmaf(c, c, m2);
+            if (left > 3) m2 = fmaf(d, d, m2);
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) dev(v[i], i0 + i * TPR);
+        for (int q = i0 + KEEP * TPR; q < nv; q += TPR) dev(__ldcg(reinterpret_cast<const float4*>(xr) + q), q);
+        auto merge = [&](float no, float mo, float so) {
+            const float t = n + no, dl = mo - mean, w = t > 0.f ? no / t : 0.f;
+            mean = fmaf(dl, w, mean);
+            m2 += so + dl * dl * n * w;
+            n = t;
+        };
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+            merge(__shfl_xor_sync(0xffffffffu, n, o), __shfl_xor_sync(0xffffffffu, mean, o), __shfl_xor_sync(0xffffffffu, m2, o));
+        if (WPR > 1) {
+            if ((threadIdx.x & 31) == 0) {
+                red[warp * 3] = n;
+                red[warp * 3 + 1] = mean;
+                red[warp * 3 + 2] = m2;
+            }
+            __syncthreads();
+            const float* p = red + r * WPR * 3;
+            n = p[0]; mean = p[1]; m2 = p[2];
+#pragma unroll
+            for (int w = 1; w < WPR; ++w) merge(p[3 * w], p[3 * w + 1], p[3 * w + 2]);
+        }
+        if (!on) return;
+        const float rstd = 1.0f / sqrtf(m2 / (float)width + eps);
+        bf16* X1 = X + (size_t)r * ld;
+        bf16* X2 = X + (size_t)(RT + r) * ld;
+        auto put = [&](const float4& u, int q) {
+            const float f[4] = {u.x, u.y, u.z, u.w};
+            float a[4], b[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int k = 4 * q + j;
+                const bool in = k < width;
+                const float d = (f[j] - mean) * rstd;
+                a[j] = in ? fmaf(d, __ldg(n1.w + k), __ldg(n1.b + k)) : 0.f;
+                b[j] = in && n2.w ? fmaf(d, __ldg(n2.w + k), __ldg(n2.b + k)) : 0.f;
+            }
+            Store<bf16>::put2(X1 + 4 * q, a[0], a[1]);
+            Store<bf16>::put2(X1 + 4 * q + 2, a[2], a[3]);
+            Store<bf16>::put2(X2 + 4 * q, b[0], b[1]);
+            Store<bf16>::put2(X2 + 4 * q + 2, b[2], b[3]);
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (4 * (i0 + i * TPR) < K) put(v[i], i0 + i * TPR);
+        for (int q = i0 + KEEP * TPR; 4 * q < K; q += TPR)
+            put(q < nv ? __ldcg(reinterpret_cast<const float4*>(xr) + q) : make_float4(0.f, 0.f, 0.f, 0.f), q);
+    }
+    __device__ __forceinline__ int tile_of(int n) const { return n >= split ? 1 : 0; }
 };
 
 // RMSNorm of an fp32 row (the queries' latent); the grid's last CTA appends the call's cache rows.
@@ -463,6 +596,51 @@ struct StageLatentQ {
     __device__ __forceinline__ void extra(int M) const {
         for (int m = threadIdx.x >> 5; m < M; m += LM_WARPS) latent_row<T>(lat, m, threadIdx.x & 31);
     }
+    static constexpr int TILES = 1;
+    static constexpr bool K_PARTS = false;
+    template <int RT>
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, int K, int M, int) const {
+        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, KEEP = 8;
+        const int r = threadIdx.x / TPR, i0 = threadIdx.x % TPR, warp = threadIdx.x >> 5;
+        const bool on = r < M;
+        const float* src = dq + (size_t)(on ? r : 0) * lddq;
+        float2 v[KEEP];
+        float ss = 0.f;
+        auto get = [&](int q) {   // elements 2q, 2q + 1 (lddq is even; past q_rank: zero)
+            float2 u = on && 2 * q < q_rank ? __ldcg(reinterpret_cast<const float2*>(src) + q) : make_float2(0.f, 0.f);
+            if (2 * q + 1 >= q_rank) u.y = 0.f;
+            return u;
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) {
+            v[i] = get(i0 + i * TPR);
+            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+        }
+        for (int q = i0 + KEEP * TPR; 2 * q < q_rank; q += TPR) {
+            const float2 u = get(q);
+            ss = fmaf(u.x, u.x, fmaf(u.y, u.y, ss));
+        }
+        ss = warp_sum(ss);
+        if (WPR > 1) {
+            if ((threadIdx.x & 31) == 0) red[warp] = ss;
+            __syncthreads();
+            ss = 0.f;
+#pragma unroll
+            for (int w = 0; w < WPR; ++w) ss += red[r * WPR + w];
+        }
+        if (!on) return;
+        const float rinv = 1.0f / sqrtf(ss / (float)q_rank + eps);
+        bf16* Xr = X + (size_t)r * ld;
+        auto put = [&](const float2& u, int q) {
+            const float w0 = 2 * q < q_rank ? __ldg(norm_w + 2 * q) : 0.f, w1 = 2 * q + 1 < q_rank ? __ldg(norm_w + 2 * q + 1) : 0.f;
+            Store<bf16>::put2(Xr + 2 * q, u.x * rinv * w0, u.y * rinv * w1);
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (2 * (i0 + i * TPR) < K) put(v[i], i0 + i * TPR);
+        for (int q = i0 + KEEP * TPR; 2 * q < K; q += TPR) put(get(q), q);
+    }
+    __device__ __forceinline__ int tile_of(int) const { return 0; }
 };
 
 template <class T>
@@ -482,7 +660,149 @@ struct StageRowsT {
     template <int RT>
     __device__ __forceinline__ const T* tile(const unsigned char* sm, int, int) const { return reinterpret_cast<const T*>(sm); }
     __device__ __forceinline__ void extra(int) const {}
+    static constexpr int TILES = 1;
+    static constexpr bool K_PARTS = true;   // may stage one CTA's part of K alone
+    template <int RT>
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float*, int K, int M, int k0) const {
+        const int nv = K / 8;
+        for (int r = 0; r < M; ++r)
+            for (int v = threadIdx.x; v < nv; v += LM_THREADS)
+                *reinterpret_cast<uint4*>(X + (size_t)r * ld + v * 8) = __ldcg(reinterpret_cast<const uint4*>(x + (size_t)r * ldx + k0) + v);
+    }
+    __device__ __forceinline__ int tile_of(int) const { return 0; }
 };
+
+struct StreamArgs {
+    const bf16* W;
+    int K, M;
+    int n_groups;     // groups of 16 weight rows
+    int kw;           // warps of a CTA along K; the CTA takes 8 / kw groups at a time
+    int ck;           // CTAs of a cluster along K (1, 2, 4), each with a contiguous part
+};
+
+template <int RT, class Stage, class Epi>
+static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Epi ep, StreamArgs a) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ float red[3 * LM_WARPS];
+    __shared__ __align__(16) float part[LM_WARPS][16][8];
+    constexpr int U = 4;       // 32-k blocks per round, two rounds in flight
+    bf16* X = reinterpret_cast<bf16*>(smem_raw);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int Kc = a.K / a.ck, ld = Kc + LS_PAD;
+    pdl_trigger();
+    if (Stage::HAS_EXTRA && blockIdx.x == gridDim.x - 1) {
+        pdl_wait();
+        st.extra(a.M);
+        return;
+    }
+    const int n_cta = (gridDim.x - (Stage::HAS_EXTRA ? 1 : 0)) / a.ck, cta = blockIdx.x / a.ck, rank = blockIdx.x % a.ck;
+    const int gpc = LM_WARPS / a.kw, gi = warp / a.kw, kp = warp % a.kw, ksplit = a.kw;
+    const int nkb = Kc / 32, my_kb = (nkb - kp + ksplit - 1) / ksplit;    // this warp's blocks: kp, kp + ksplit, ...
+    const int rounds = ((nkb + ksplit - 1) / ksplit + U - 1) / U;            // the same for every warp
+    const int sets = (a.n_groups + gpc * n_cta - 1) / (gpc * n_cta);
+    uint4 w0[2][U], w1[2][U];
+    // round it of set s: weight rows g and g + 8 of the group, 8 consecutive k per lane and block
+    auto load = [&](int buf, int s, int it) {
+        const int grp = (s * n_cta + cta) * gpc + gi;
+        const bool live = grp < a.n_groups;
+        const bf16* p = a.W + (size_t)((live ? grp : 0) * 16 + g) * a.K + rank * Kc + t * 8;
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int b = it * U + u;
+            const bool ok = live && b < my_kb;
+            const size_t o = (size_t)(kp + b * ksplit) * 32;
+            w0[buf][u] = ok ? ldg_stream(p + o) : make_uint4(0, 0, 0, 0);
+            w1[buf][u] = ok ? ldg_stream(p + (size_t)8 * a.K + o) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    const int total = sets * rounds;
+    load(0, 0, 0);
+    if (total > 1) load(1, rounds > 1 ? 0 : 1, rounds > 1 ? 1 : 0);
+    pdl_wait();
+    st.template stage_rows<RT>(X, ld, red, Kc, a.M, rank * Kc);
+    __syncthreads();
+    const int xrow = min(g, a.M - 1);   // columns past the last row repeat it and are not stored
+    int s = 0, it = 0;
+    float acc[2][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[0][i] = acc[1][i] = 0.f;
+    auto round = [&](int buf, int i) {
+        if (it == 0)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) acc[0][c] = acc[1][c] = 0.f;
+        const int grp = (s * n_cta + cta) * gpc + gi;
+        const bf16* xp = X + (size_t)(Stage::TILES > 1 ? st.tile_of(grp * 16) * RT : 0) * ld + (size_t)xrow * ld + t * 8;
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int b = it * U + u;
+            if (b < my_kb) {
+                const uint4 x = *reinterpret_cast<const uint4*>(xp + (size_t)(kp + b * ksplit) * 32);
+                const uint32_t a0[4] = {w0[buf][u].x, w1[buf][u].x, w0[buf][u].y, w1[buf][u].y};
+                const uint32_t a1[4] = {w0[buf][u].z, w1[buf][u].z, w0[buf][u].w, w1[buf][u].w};
+                asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                             : "+f"(acc[0][0]), "+f"(acc[0][1]), "+f"(acc[0][2]), "+f"(acc[0][3])
+                             : "r"(a0[0]), "r"(a0[1]), "r"(a0[2]), "r"(a0[3]), "r"(x.x), "r"(x.y));
+                asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                             : "+f"(acc[1][0]), "+f"(acc[1][1]), "+f"(acc[1][2]), "+f"(acc[1][3])
+                             : "r"(a1[0]), "r"(a1[1]), "r"(a1[2]), "r"(a1[3]), "r"(x.z), "r"(x.w));
+            }
+        }
+        // two rounds ahead
+        if (i + 2 < total) {
+            int s2 = s, it2 = it + 2;
+            while (it2 >= rounds) { it2 -= rounds; ++s2; }
+            load(buf, s2, it2);
+        }
+        if (++it < rounds) return;
+        it = 0;
+        // the set is complete: sums meet in shared memory
+        *reinterpret_cast<float2*>(&part[warp][g][2 * t]) = make_float2(acc[0][0] + acc[1][0], acc[0][1] + acc[1][1]);
+        *reinterpret_cast<float2*>(&part[warp][g + 8][2 * t]) = make_float2(acc[0][2] + acc[1][2], acc[0][3] + acc[1][3]);
+        if (a.ck > 1) {
+            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        } else {
+            __syncthreads();
+        }
+        // 8 pairs of rows per group x M rows, dealt to the threads of the CTA (of the cluster)
+        const int base = (s * n_cta + cta) * gpc;
+        const int n_out = gpc * 8 * a.M;
+        for (int o = rank * LM_THREADS + threadIdx.x; o < n_out; o += a.ck * LM_THREADS) {
+            const int pr = o % 8, gm = o / 8, q = gm % gpc, m = gm / gpc;
+            if (base + q >= a.n_groups) continue;
+            float v0 = 0.f, v1 = 0.f;
+            for (int c = 0; c < a.ck; ++c) {
+                for (int w = 0; w < a.kw; ++w) {
+                    const float* p = &part[q * a.kw + w][2 * pr][m];
+                    if (a.ck == 1) {
+                        v0 += p[0];
+                        v1 += p[8];
+                    } else {
+                        uint32_t ra;
+                        float f0, f1;
+                        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(c));
+                        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(f0) : "r"(ra) : "memory");
+                        asm volatile("ld.shared::cluster.f32 %0, [%1 + 32];" : "=f"(f1) : "r"(ra) : "memory");
+                        v0 += f0;
+                        v1 += f1;
+                    }
+                }
+            }
+            ep.store(m, (base + q) * 16 + 2 * pr, v0, v1);
+        }
+        if (a.ck > 1) {   // no CTA leaves while a peer may still read its sums
+            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        } else if (s + 1 < sets) {
+            __syncthreads();
+        }
+        ++s;
+    };
+    for (int i = 0; i < total; i += 2) {
+        round(0, i);
+        if (i + 1 < total) round(1, i + 1);
+    }
+}
 
 template <class T, int RT, class Stage, class Epi>
 static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_gemv(Stage st, Epi ep, const T* __restrict__ W, int K, int M,
