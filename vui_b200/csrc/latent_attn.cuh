@@ -67,15 +67,16 @@ struct LatentAttnArgs {
     const void* cache;        // (n_slots, max_seq, Dp) T of this layer
     const int32_t* row_slot;
     const int32_t* row_pos;
-    int H, Rp, Dp, max_seq;
+    int H, Rp, Dp, max_seq, n_slots;
     int nbuf;                 // key tiles in shared memory (1 or 2)
     float scale;
-    FastDiv row_vecs;         // Dp / 8
+    FastDiv row_vecs, w_vecs; // Dp / 8, Rp / 8
     // bf16: value matrix and gate (fused), or the latent sums (M, H, Rp)
     const bf16* wuv;          // (H, vdim, Rp)
     const bf16* gate;         // (M, ldgate)
     bf16* out;                // fused: (M, ldo) gated values; else the latent sums
     int ldgate, ldo, vdim;
+    int w_smem;               // fused: the CTA's value matrices are brought to shared memory before the dependency wait
     // fp32: partial sums of the splits
     float* part;              // (M, S, H, Rp)
     float* ml;                // (M, S, H, 2): running maximum and sum
@@ -92,29 +93,12 @@ __device__ __forceinline__ void latent_splits(int len, int keys, int S, int& tps
 
 constexpr int LA_MAX_CL = 8;      // CTAs (key splits) of a row's cluster
 
-static inline size_t latent_attn_smem(int Dp, int Rp, int nbuf, int fuse_heads = 0) {
+// fuse_heads: heads a CTA finishes itself (0: it does not); w_rows: rows of the value matrices it keeps
+static inline size_t latent_attn_smem(int Dp, int Rp, int nbuf, int fuse_heads = 0, int w_rows = 0) {
     const size_t keys = (size_t)nbuf * LA_KEYS * (Dp + 8) * 2, sums = (size_t)16 * (Rp + 4) * 4;   // share their space
     return (size_t)16 * (Dp + 8) * 2 + (keys > sums ? keys : sums) + 16 * (LA_KEYS + 4) * 4 + 2 * 16 * (LA_KEYS + 8) * 2 +
-           16 * 4 + 16 * 8 + (size_t)fuse_heads * Rp * 4;
+           16 * 4 + 16 * 8 + (size_t)fuse_heads * Rp * 2 + (size_t)w_rows * (Rp + LS_PAD) * 2;
 }
-
-__device__ __forceinline__ uint32_t cluster_addr(const void* p, int rank) {
-    uint32_t ra;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(rank));
-    return ra;
-}
-__device__ __forceinline__ float ld_cluster(uint32_t a) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
-    return v;
-}
-__device__ __forceinline__ float2 ld_cluster2(uint32_t a) {
-    float2 v;
-    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(a) : "memory");
-    return v;
-}
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 
 // One cluster of CL CTAs per (query row, 16 heads): CTA = a split of the keys.  The CTAs leave their partial sums in
 // shared memory; each then merges 16 / CL heads over the cluster in split order, and either writes the latent sums or
@@ -138,10 +122,24 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     const int sp = blockIdx.x % CL, hg = blockIdx.x / CL, m = blockIdx.y;
     const int hpc = 16 / CL, h_loc0 = sp * hpc, h0 = hg * 16 + h_loc0;   // heads this CTA finishes
     const int n_fin = max(0, min(hpc, a.H - h0));
-    if constexpr (FUSE_V) {   // the value matrices are constants: on their way to L2 while the predecessor runs
-        const char* p = reinterpret_cast<const char*>(a.wuv + (size_t)h0 * a.vdim * a.Rp);
-        for (size_t i = (size_t)tid * 128; i < (size_t)n_fin * a.vdim * a.Rp * 2; i += LM_THREADS * 128)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(p + i));
+    bf16* ol = reinterpret_cast<bf16*>(ml_s + 32);      // [hpc][Rp] merged sums (FUSE_V)
+    bf16* Ws = ol + (FUSE_V ? hpc * a.Rp : 0);          // [n_fin * vdim][Rp + LS_PAD] (FUSE_V, w_smem)
+    if constexpr (FUSE_V) {   // the value matrices are constants: on their way while the predecessor runs
+        const bf16* p = a.wuv + (size_t)h0 * a.vdim * a.Rp;
+        const int n = n_fin * a.vdim * a.Rp;            // a multiple of 16
+        if (a.w_smem) {
+            for (int i = tid; i < n / 8; i += LM_THREADS) cp_async16(Ws + i * 8 + a.w_vecs.div(i) * LS_PAD, p + i * 8, true);
+            cp_async_commit();
+        } else {
+            for (int i = tid * 64; i < n; i += LM_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + i));
+        }
+        // The rows of this split, as the table reads now, on their way to L2: a hint only, read again below.
+        const int s_ = min(max(__ldcg(a.row_slot + m), 0), a.n_slots - 1), l_ = min(max(__ldcg(a.row_pos + m), 0), a.max_seq - 1);
+        int tps, ns;
+        latent_splits(l_ + 1, LA_KEYS, CL, tps, ns);
+        const bf16* kb = static_cast<const bf16*>(a.cache) + (size_t)s_ * a.max_seq * a.Dp;
+        const int e0 = min(l_, sp * tps * LA_KEYS) * a.Dp, e1 = min(l_, min((sp + 1) * tps, sp * tps + 4) * LA_KEYS) * a.Dp;
+        for (int i = e0 + tid * 64; i < e1; i += LM_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(kb + i));
     }
     pdl_wait();
     const int slot = __ldcg(a.row_slot + m), len = __ldcg(a.row_pos + m) + 1;
@@ -185,7 +183,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
         const bf16* qp = Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
         const bf16* kp = K + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
         int ks = 0;
-#pragma unroll 4
+#pragma unroll 2
         for (; ks + 2 <= ksteps; ks += 2) {
             uint32_t a0[4], a1[4], b[4];
             ldsm_x4(a0, qp + ks * 16);
@@ -234,8 +232,8 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
             acc[i][0] *= c_lo; acc[i][1] *= c_lo;
             acc[i][2] *= c_hi; acc[i][3] *= c_hi;
         }
-#pragma unroll
-        for (int j = 0; j < LA_KEYS / 16; ++j) {
+#pragma unroll 1
+        for (int j = 0; j < LA_KEYS / 16 && j * 16 < left; ++j) {
             uint32_t ph[4], pl[4];
             const int po = ((lane & 7) + ((lane >> 3) & 1) * 8) * PP + j * 16 + (lane >> 4) * 8;
             ldsm_x4(ph, Ph + po);
@@ -256,6 +254,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
         __syncthreads();   // the tile and the weights are used up
         if (!ahead && tile + 1 < n_tiles) fetch(tile + 1);
     }
+    if (FUSE_V && n_tiles == 0) cp_async_wait<0>();      // the value matrices
     // ---- partial sums, maxima and totals for the cluster
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
@@ -272,7 +271,6 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     cluster_wait();
     // ---- merge: 256 / hpc threads per head
     const int tph = LM_THREADS / hpc, hl = tid / tph, c0 = tid % tph;
-    float* ol = ml_s + 32;                              // [hpc][Rp] merged sums (FUSE_V)
     if (hl < n_fin) {
         float w[LA_MAX_CL], mx = NEG_BIG, l = 0.f;
         float2 p[LA_MAX_CL];
@@ -292,7 +290,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
 #pragma unroll
             for (int s = 0; s < LA_MAX_CL; ++s)
                 if (s < ns) o = fmaf(w[s], ld_cluster(cluster_addr(Os + (h_loc0 + hl) * lds + c, s)), o);
-            if constexpr (FUSE_V) ol[hl * a.Rp + c] = o * inv;
+            if constexpr (FUSE_V) ol[hl * a.Rp + c] = f2bf(o * inv);
             else a.out[((size_t)m * a.H + h0 + hl) * a.Rp + c] = f2bf(o * inv);
         }
     }
@@ -300,30 +298,37 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     cluster_arrive();
     if constexpr (FUSE_V) {
         __syncthreads();
-        // rows (head, d) of the value matrices, four at a time per warp
-        const int n_rows = n_fin * a.vdim, nvr = a.Rp / 8;
-        const bf16* W = a.wuv + (size_t)h0 * a.vdim * a.Rp;
-        for (int r0 = warp * 4; r0 < n_rows; r0 += LM_WARPS * 4) {
-            float s[4] = {0.f, 0.f, 0.f, 0.f};
-            for (int v = lane; v < nvr; v += 32) {
-                uint4 w[4];
-#pragma unroll
-                for (int u = 0; u < 4; ++u) w[u] = ldg_stream(W + (size_t)min(r0 + u, n_rows - 1) * a.Rp + v * 8);
-#pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const float* o = ol + (min(r0 + u, n_rows - 1) / a.vdim) * a.Rp + v * 8;
-                    float f[8];
-                    unpack8(w[u], f);
-                    const float4 x = *reinterpret_cast<const float4*>(o), y = *reinterpret_cast<const float4*>(o + 4);
-                    s[u] = fmaf(f[0], x.x, fmaf(f[1], x.y, fmaf(f[2], x.z, fmaf(f[3], x.w, s[u]))));
-                    s[u] = fmaf(f[4], y.x, fmaf(f[5], y.y, fmaf(f[6], y.z, fmaf(f[7], y.w, s[u]))));
-                }
+        // 16 value rows of a head per warp (the M side), k in the lanes' own order as in k_lm_stream; the N side is this row
+        const int gph = (a.vdim + 15) / 16, blocks = (a.Rp + 31) / 32, nkb = a.Rp / 32;
+        const size_t wst = a.w_smem ? a.Rp + LS_PAD : a.Rp;
+        const bf16* W = a.w_smem ? Ws : a.wuv + (size_t)h0 * a.vdim * a.Rp;
+        for (int q = warp; q < n_fin * gph; q += LM_WARPS) {
+            const int h = q / gph, d0 = (q - h * gph) * 16;
+            const int d_lo = d0 + g, d_hi = d0 + g + 8;
+            const bf16* w0 = W + ((size_t)h * a.vdim + min(d_lo, a.vdim - 1)) * wst + t * 8;
+            const bf16* w1 = W + ((size_t)h * a.vdim + min(d_hi, a.vdim - 1)) * wst + t * 8;
+            const bf16* o = ol + h * a.Rp + t * 8;
+            const size_t col = (size_t)(h0 + h) * a.vdim;
+            float g_lo = 0.f, g_hi = 0.f;
+            if (t == 0) {
+                if (d_lo < a.vdim) g_lo = bf2f(a.gate[(size_t)m * a.ldgate + col + d_lo]);
+                if (d_hi < a.vdim) g_hi = bf2f(a.gate[(size_t)m * a.ldgate + col + d_hi]);
             }
-#pragma unroll
-            for (int u = 0; u < 4; ++u) s[u] = warp_sum(s[u]);
-            if (lane < 4 && r0 + lane < n_rows) {
-                const size_t c = (size_t)h0 * a.vdim + r0 + lane;
-                a.out[(size_t)m * a.ldo + c] = f2bf(pick<4>(s, lane) * bf2f(a.gate[(size_t)m * a.ldgate + c]));
+            float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+            for (int b = 0; b < blocks; ++b) {
+                const bool in = b < nkb || t < 2;        // lanes 2, 3 of a half block hold zeros
+                const uint4 z = make_uint4(0, 0, 0, 0);
+                const uint4 x0 = in ? *reinterpret_cast<const uint4*>(w0 + b * 32) : z, x1 = in ? *reinterpret_cast<const uint4*>(w1 + b * 32) : z;
+                const uint4 y = in ? *reinterpret_cast<const uint4*>(o + b * 32) : z;
+                const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
+                mma_bf16(c0, a0, y.x, y.y);
+                mma_bf16(c1, a1, y.z, y.w);
+            }
+            if (t == 0) {                                // every column holds the same sums: column 0 is this lane's
+                bf16* dst = a.out + (size_t)m * a.ldo + col;
+                if (d_lo < a.vdim) dst[d_lo] = f2bf((c0[0] + c1[0]) * g_lo);
+                if (d_hi < a.vdim) dst[d_hi] = f2bf((c0[2] + c1[2]) * g_hi);
             }
         }
     }
@@ -331,7 +336,8 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
 }
 
 // Many rows: out[m][h*vdim + d] = gate * sum_k W_uv[h][d][k] o[m][h][k] as one small product per head.  A warp owns 16
-// value rows (the M side) and 32 activation rows (the N side); k is taken in the lanes' own order as in k_lm_stream.
+// value rows (the M side) and 16 activation rows (the N side); k is taken in the lanes' own order as in k_lm_stream.
+constexpr int LV_TILES = 2;
 struct LatentValueArgs {
     const bf16* wuv;       // (H, vdim, Rp)
     const bf16* o;         // (M, H, Rp)
@@ -343,32 +349,43 @@ struct LatentValueArgs {
 static __global__ void __launch_bounds__(128) k_latent_value(LatentValueArgs a) {
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    const int h = blockIdx.x, d0 = (blockIdx.y * 4 + warp) * 16, m0 = blockIdx.z * 32;
+    const int h = blockIdx.x, d0 = (blockIdx.y * 4 + warp) * 16, m0 = blockIdx.z * 8 * LV_TILES;
     const int nkb = a.Rp / 32;                       // Rp is a multiple of 16: a half block may be left
     const bf16* w0 = a.wuv + ((size_t)h * a.vdim + min(d0 + g, a.vdim - 1)) * a.Rp + t * 8;
     const bf16* w1 = a.wuv + ((size_t)h * a.vdim + min(d0 + g + 8, a.vdim - 1)) * a.Rp + t * 8;
-    const bf16* o[4];
+    const bf16* o[LV_TILES];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) o[j] = a.o + ((size_t)min(m0 + j * 8 + g, a.M - 1) * a.H + h) * a.Rp + t * 8;
-    float acc[4][4];
+    for (int j = 0; j < LV_TILES; ++j) o[j] = a.o + ((size_t)min(m0 + j * 8 + g, a.M - 1) * a.H + h) * a.Rp + t * 8;
+    float acc[LV_TILES][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int j = 0; j < LV_TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     pdl_wait();
     if (d0 >= a.vdim) return;
     const int blocks = (a.Rp + 31) / 32;
-    for (int b = 0; b < blocks; ++b) {
-        const bool in = b < nkb || t < 2;            // lanes 2, 3 of a half block hold zeros
-        const uint4 x0 = in ? ldg_stream(w0 + b * 32) : make_uint4(0, 0, 0, 0), x1 = in ? ldg_stream(w1 + b * 32) : make_uint4(0, 0, 0, 0);
-        const uint32_t a0[4] = {x0.x, x1.x, x0.y, x1.y}, a1[4] = {x0.z, x1.z, x0.w, x1.w};
+    constexpr int U = 4;     // blocks requested together
+    for (int b0 = 0; b0 < blocks; b0 += U) {
+        uint4 x0[U], x1[U], y[U][LV_TILES];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const uint4 y = in ? __ldcg(reinterpret_cast<const uint4*>(o[j] + b * 32)) : make_uint4(0, 0, 0, 0);
-            mma_bf16(acc[j], a0, y.x, y.y);
-            mma_bf16(acc[j], a1, y.z, y.w);
+        for (int u = 0; u < U; ++u) {
+            const int b = b0 + u;
+            const bool in = b < nkb || (b < blocks && t < 2);   // lanes 2, 3 of a half block hold zeros
+            x0[u] = in ? ldg_stream(w0 + b * 32) : make_uint4(0, 0, 0, 0);
+            x1[u] = in ? ldg_stream(w1 + b * 32) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+            for (int j = 0; j < LV_TILES; ++j) y[u][j] = in ? __ldcg(reinterpret_cast<const uint4*>(o[j] + b * 32)) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const uint32_t a0[4] = {x0[u].x, x1[u].x, x0[u].y, x1[u].y}, a1[4] = {x0[u].z, x1[u].z, x0[u].w, x1[u].w};
+#pragma unroll
+            for (int j = 0; j < LV_TILES; ++j) {
+                mma_bf16(acc[j], a0, y[u][j].x, y[u][j].y);
+                mma_bf16(acc[j], a1, y[u][j].z, y[u][j].w);
+            }
         }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < LV_TILES; ++j)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const int d = d0 + g + (c >> 1) * 8, m = m0 + j * 8 + 2 * t + (c & 1);

@@ -29,7 +29,11 @@ namespace {
 constexpr int LM_FEW_ROWS = 8;         // rows up to which the weight-streaming products run (fp32: 4)
 constexpr int LM_FEW_ROWS_F32 = 4;
 constexpr int LA_ROW_BLOCK = 512;      // rows of one fp32 attention launch (bounds the split scratch)
-constexpr int LA_CTAS = 2 * 148;       // CTAs of one wave: what rows of weights and splits of keys are cut to
+constexpr int LA_CTAS = 2 * 148;       // CTAs the key splits are cut to
+// CTAs of a streaming product: one per SM, so that the next kernel's fit beside them and request their weights early;
+// two for a matrix of which the next kernel's early requests are a small part.
+constexpr int LS_CTAS = 148;
+constexpr size_t LS_LARGE = (size_t)48 << 20;
 constexpr int LM_EXPAND_MIN = 64;      // rows of a call from which a prefill expands keys and values
 constexpr size_t LM_MAX_SMEM = 227 * 1024;
 
@@ -240,11 +244,13 @@ constexpr size_t LS_MAX_SMEM = 200 * 1024;
 // CTAs of a cluster along K for a product whose rows alone do not fill the SMs.
 int stream_ck(int n_groups, int K, bool k_parts) {
     int ck = 1;
-    while (k_parts && ck < 4 && n_groups * ck * 2 <= LA_CTAS && K % (64 * ck) == 0 && K / (2 * ck) >= 256) ck *= 2;
+    if ((size_t)n_groups * 32 * K > LS_LARGE) return 1;
+    while (k_parts && ck < 4 && n_groups * ck * 2 <= LS_CTAS && K % (64 * ck) == 0 && K / (2 * ck) >= 256) ck *= 2;
     return ck;
 }
 
-size_t stream_smem(int tiles, int rt, int K, int ck) { return (size_t)tiles * rt * (K / ck + LS_PAD) * 2; }
+template <class Stage>
+size_t stream_smem(int rt, int K, int ck) { return (size_t)Stage::TILES * rt * (K / ck + LS_PAD) * 2 + Stage::scratch(rt, K); }
 
 template <int RT, class Stage, class Epi>
 int32_t stream_rt(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int K, int M, int n_rows, cudaStream_t s) {
@@ -256,12 +262,12 @@ int32_t stream_rt(VuibLm* e, const Stage& st, const Epi& ep, const void* W, int 
     a.ck = stream_ck(a.n_groups, K, Stage::K_PARTS);
     // warps along K: as many as the one wave of CTAs has to spare, two 32-k blocks each at least
     a.kw = 1;
-    const int blocks = K / a.ck / 32;
-    while (a.kw < LM_WARPS && a.n_groups * a.ck * a.kw * 2 <= LA_CTAS * LM_WARPS && a.kw * 4 <= blocks) a.kw *= 2;
-    const int gpc = LM_WARPS / a.kw, need = (a.n_groups + gpc - 1) / gpc, most = LA_CTAS / a.ck;
+    const int blocks = K / a.ck / 32, wave = (size_t)n_rows * K * 2 > LS_LARGE ? 2 * LS_CTAS : LS_CTAS;
+    while (a.kw < LM_WARPS && a.n_groups * a.ck * a.kw * 2 <= wave * LM_WARPS && a.kw * 4 <= blocks) a.kw *= 2;
+    const int gpc = LM_WARPS / a.kw, need = (a.n_groups + gpc - 1) / gpc, most = wave / a.ck;
     const int sets = (need + most - 1) / most, ctas = (need + sets - 1) / sets;
     return run_cl(e, k_lm_stream<RT, Stage, Epi>, dim3(ctas * a.ck + (Stage::HAS_EXTRA ? 1 : 0)), a.ck, LM_THREADS,
-                  stream_smem(Stage::TILES, RT, K, a.ck), s, st, ep, a);
+                  stream_smem<Stage>(RT, K, a.ck), s, st, ep, a);
 }
 
 template <int RT, class Stage, class Epi>
@@ -298,8 +304,9 @@ int few_rows_of(const VuibLm* e) {
         bool ok = true;
         for (const VuibLmDims& d : e->dims) {
             if (b16) {
-                ok = ok && stream_smem(2, rt, d.k_in, 1) <= LS_MAX_SMEM && stream_smem(1, rt, d.k_q, 1) <= LS_MAX_SMEM &&
-                     stream_smem(1, rt, d.k_out, stream_ck(up(c.width, 16) / 16, d.k_out, true)) <= LS_MAX_SMEM;
+                ok = ok && stream_smem<StageLayerNorm2<bf16>>(rt, d.k_in, 1) <= LS_MAX_SMEM &&
+                     stream_smem<StageLatentQ<bf16>>(rt, d.k_q, 1) <= LS_MAX_SMEM &&
+                     stream_smem<StageRowsT<bf16>>(rt, d.k_out, stream_ck(up(c.width, 16) / 16, d.k_out, true)) <= LS_MAX_SMEM;
             } else {   // one row at a time will do
                 ok = ok && StageLayerNorm2<float>::smem(1, d.k_in) <= LS_MAX_SMEM && StageRowsT<float>::smem(1, d.k_out) <= LS_MAX_SMEM &&
                      StageRowsT<float>::smem(1, d.k_q) <= LS_MAX_SMEM;
@@ -344,15 +351,17 @@ LatentAttnArgs attn_args(VuibLm* e, int li) {
     a.Rp = d.rp;
     a.Dp = d.dp;
     a.max_seq = e->cfg.max_seq;
+    a.n_slots = e->cfg.n_slots;
     a.scale = l.scale;
     a.row_vecs = FastDiv(d.dp / 8);
+    a.w_vecs = FastDiv(d.rp / 8);
     return a;
 }
 
 template <bool FUSE_V>
 int32_t latent_attn_nt(VuibLm* e, const LatentAttnArgs& a, int CL, int M, cudaStream_t s) {
     const dim3 grid(CL * ((a.H + 15) / 16), M);
-    const size_t sm = latent_attn_smem(a.Dp, a.Rp, a.nbuf, FUSE_V ? 16 / CL : 0);
+    const size_t sm = latent_attn_smem(a.Dp, a.Rp, a.nbuf, FUSE_V ? 16 / CL : 0, FUSE_V && a.w_smem ? 16 / CL * a.vdim : 0);
     if (a.Rp <= 128) return run_cl(e, k_latent_attn<2, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
     if (a.Rp <= 256) return run_cl(e, k_latent_attn<4, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
     if (a.Rp <= 512) return run_cl(e, k_latent_attn<8, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
@@ -376,12 +385,13 @@ int32_t absorbed_attention_bf16(VuibLm* e, int li, int M, cudaStream_t s) {
     a.ldo = L.ld_ay;
     if (M <= LM_FEW_ROWS) {
         a.out = wsp<bf16>(e, L.ay);
+        a.w_smem = latent_attn_smem(d.dp, d.rp, a.nbuf, 16 / CL, 16 / CL * l.vdim) <= 180 * 1024;
         return latent_attn_nt<true>(e, a, CL, M, s);
     }
     a.out = wsp<bf16>(e, L.olat);
     RC(latent_attn_nt<false>(e, a, CL, M, s));
     const LatentValueArgs v{a.wuv, wsp<bf16>(e, L.olat), a.gate, L.ld_gate, wsp<bf16>(e, L.ay), L.ld_ay, l.heads, d.rp, l.vdim, M};
-    return run(e, k_latent_value, dim3(l.heads, (l.vdim + 63) / 64, (M + 31) / 32), 128, 0, s, v);
+    return run(e, k_latent_value, dim3(l.heads, (l.vdim + 63) / 64, (M + 8 * LV_TILES - 1) / (8 * LV_TILES)), 128, 0, s, v);
 }
 
 int32_t absorbed_attention_f32(VuibLm* e, int li, int M, cudaStream_t s) {

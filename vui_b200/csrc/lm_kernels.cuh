@@ -59,6 +59,25 @@ __device__ __forceinline__ void block_sums(float (&v)[N], float* red) {
     }
 }
 
+// Another CTA's shared memory, and the cluster's barrier.
+__device__ __forceinline__ uint32_t cluster_addr(const void* p, int rank) {
+    uint32_t ra;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(rank));
+    return ra;
+}
+__device__ __forceinline__ float ld_cluster(uint32_t a) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
+    return v;
+}
+__device__ __forceinline__ float2 ld_cluster2(uint32_t a) {
+    float2 v;
+    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(a) : "memory");
+    return v;
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
 // Rotation of the pair (u, v) by the angle whose (cos, sin) is cs.
 __device__ __forceinline__ float2 rotate_pair(float u, float v, float2 cs) {
     return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
@@ -204,29 +223,50 @@ struct LatentRow {
 
 template <class T>
 __device__ __forceinline__ void latent_row(const LatentRow& a, int m, int lane) {
+    constexpr int KEEP = 8;       // elements of a lane held in registers, all requested together
     const float* src = a.dkv + (size_t)m * a.Dp;
     const int slot = __ldcg(a.row_slot + m), pos = __ldcg(a.row_pos + m);
-    float ss = 0.f;
-    for (int k = lane; k < a.R; k += 32) {
-        const float v = __ldcg(src + k);
-        ss = fmaf(v, v, ss);
+    float v[KEEP], w[KEEP], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int k = lane + 32 * i;
+        v[i] = k < a.R ? __ldcg(src + k) : 0.f;
+        w[i] = k < a.R ? __ldg(a.norm_w + k) : 0.f;
+    }
+    const bool one = lane * 2 + 1 < a.rot;    // the first 64 rotated components
+    float2 rv = one ? __ldcg(reinterpret_cast<const float2*>(src + a.Rp) + lane) : make_float2(0.f, 0.f);
+    T* dst = static_cast<T*>(a.cache) + ((size_t)slot * a.max_seq + pos) * a.Dp;
+    const float2* tr = a.trig + (size_t)pos * (a.rot_dims / 2);
+    const float2 cs = 2 * lane < a.rot_dims ? __ldg(tr + lane) : make_float2(1.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) ss = fmaf(v[i], v[i], ss);
+    for (int k = lane + 32 * KEEP; k < a.R; k += 32) {
+        const float u = __ldcg(src + k);
+        ss = fmaf(u, u, ss);
     }
     ss = warp_sum(ss);
     const float rinv = 1.0f / sqrtf(ss / (float)a.R + a.eps);
-    T* dst = static_cast<T*>(a.cache) + ((size_t)slot * a.max_seq + pos) * a.Dp;
-    for (int k = lane; k < a.R; k += 32) Store<T>::put(dst + k, __ldcg(src + k) * rinv * __ldg(a.norm_w + k));
-    const float2* tr = a.trig + (size_t)pos * (a.rot_dims / 2);
-    for (int i = lane; 2 * i < a.rot; i += 32) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (lane + 32 * i < a.R) Store<T>::put(dst + lane + 32 * i, v[i] * rinv * w[i]);
+    for (int k = lane + 32 * KEEP; k < a.R; k += 32) Store<T>::put(dst + k, __ldcg(src + k) * rinv * __ldg(a.norm_w + k));
+    if (one) {
+        rv = rotate_pair(rv.x, rv.y, cs);
+        Store<T>::put2(dst + a.Rp + 2 * lane, rv.x, rv.y);
+    } else if (lane * 2 < a.rot) {            // an odd component at the end is never rotated
+        Store<T>::put(dst + a.Rp + 2 * lane, __ldcg(src + a.Rp + 2 * lane));
+    }
+    for (int i = lane + 32; 2 * i < a.rot; i += 32) {
         float u = __ldcg(src + a.Rp + 2 * i);
         const bool pair = 2 * i + 1 < a.rot;
-        float v = pair ? __ldcg(src + a.Rp + 2 * i + 1) : 0.f;
+        float x = pair ? __ldcg(src + a.Rp + 2 * i + 1) : 0.f;
         if (2 * i < a.rot_dims) {
-            const float2 o = rotate_pair(u, v, __ldg(tr + i));
+            const float2 o = rotate_pair(u, x, __ldg(tr + i));
             u = o.x;
-            v = o.y;
+            x = o.y;
         }
         Store<T>::put(dst + a.Rp + 2 * i, u);
-        if (pair) Store<T>::put(dst + a.Rp + 2 * i + 1, v);
+        if (pair) Store<T>::put(dst + a.Rp + 2 * i + 1, x);
     }
 }
 
@@ -472,89 +512,80 @@ struct StageLayerNorm2 {
     __device__ __forceinline__ void extra(int) const {}
     static constexpr bool HAS_EXTRA = false;
 
-    // k_lm_stream form: 8 / RT warps per row; (count, mean, sum of squared deviations) of the pieces are merged, so
-    // that one exchange gives mean and variance
+    // k_lm_stream form: 8 / RT warps per row.  The norms' vectors are constants and come to shared memory before the
+    // dependency wait; the row is kept there in 32 bits between the passes.
     static constexpr int TILES = 2;
     static constexpr bool K_PARTS = false;
+    static __host__ __device__ size_t scratch(int RT, int K) { return (size_t)(RT + 4) * K * 4; }
+    __device__ __forceinline__ void constants(float* sc, int K) const {
+        const float* src[4] = {n1.w, n1.b, n2.w, n2.b};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (src[i])
+                for (int k = threadIdx.x; k < width; k += LM_THREADS) sc[i * K + k] = __ldg(src[i] + k);
+    }
     template <int RT>
-    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, int K, int M, int) const {
-        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, KEEP = 4;
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, float* sc, int K, int M, int) const {
+        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, U = 4;
         const int r = threadIdx.x / TPR, i0 = threadIdx.x % TPR, warp = threadIdx.x >> 5;
         const bool on = r < M;
         const float* xr = x + (size_t)(on ? (rows ? rows[r] : r) : 0) * ldx;
-        const int nv = (width + 3) / 4;    // ldx is a multiple of 64 and the row's pad is zero
-        float4 v[KEEP];
-        float n = 0.f, mean = 0.f, m2 = 0.f;
+        float* xs = sc + (size_t)(4 + r) * K;
+        const int nv = K / 4;              // K = ldx, and the row's pad is zero
+        float sum = 0.f;
+        for (int q0 = i0; q0 < nv; q0 += U * TPR) {
+            float4 v[U];
 #pragma unroll
-        for (int i = 0; i < KEEP; ++i) {
-            const int q = i0 + i * TPR;
-            v[i] = on && q < nv ? __ldcg(reinterpret_cast<const float4*>(xr) + q) : make_float4(0.f, 0.f, 0.f, 0.f);
-            mean += (v[i].x + v[i].y) + (v[i].z + v[i].w);
-            n += (float)max(0, min(4, width - 4 * q));
+            for (int u = 0; u < U; ++u)
+                v[u] = q0 + u * TPR < nv ? __ldcg(reinterpret_cast<const float4*>(xr) + q0 + u * TPR) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+                if (q0 + u * TPR < nv) {
+                    reinterpret_cast<float4*>(xs)[q0 + u * TPR] = v[u];
+                    sum += (v[u].x + v[u].y) + (v[u].z + v[u].w);
+                }
         }
-        for (int q = i0 + KEEP * TPR; q < nv; q += TPR) {
-            const float4 u = __ldcg(reinterpret_cast<const float4*>(xr) + q);
-            mean += (u.x + u.y) + (u.z + u.w);
-            n += (float)min(4, width - 4 * q);
-        }
-        mean = n > 0.f ? mean / n : 0.f;
-        auto dev = [&](const float4& u, int q) {
-            const float a = u.x - mean, b = u.y - mean, c = u.z - mean, d = u.w - mean;
-            const int left = width - 4 * q;
-            if (left > 0) m2 = fmaf(a, a, m2);
-            if (left > 1) m2 = fmaf(b, b, m2);
-            if (left > 2) m2 = fmaf(c, c, m2);
-            if (left > 3) m2 = fmaf(d, d, m2);
-        };
+        auto row_total = [&](float t, float* buf) {
+            t = warp_sum(t);
+            if (WPR > 1) {
+                if ((threadIdx.x & 31) == 0) buf[warp] = t;
+                __syncthreads();
+                t = 0.f;
 #pragma unroll
-        for (int i = 0; i < KEEP; ++i) dev(v[i], i0 + i * TPR);
-        for (int q = i0 + KEEP * TPR; q < nv; q += TPR) dev(__ldcg(reinterpret_cast<const float4*>(xr) + q), q);
-        auto merge = [&](float no, float mo, float so) {
-            const float t = n + no, dl = mo - mean, w = t > 0.f ? no / t : 0.f;
-            mean = fmaf(dl, w, mean);
-            m2 += so + dl * dl * n * w;
-            n = t;
-        };
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1)
-            merge(__shfl_xor_sync(0xffffffffu, n, o), __shfl_xor_sync(0xffffffffu, mean, o), __shfl_xor_sync(0xffffffffu, m2, o));
-        if (WPR > 1) {
-            if ((threadIdx.x & 31) == 0) {
-                red[warp * 3] = n;
-                red[warp * 3 + 1] = mean;
-                red[warp * 3 + 2] = m2;
+                for (int w = 0; w < WPR; ++w) t += buf[r * WPR + w];
             }
-            __syncthreads();
-            const float* p = red + r * WPR * 3;
-            n = p[0]; mean = p[1]; m2 = p[2];
+            return t;
+        };
+        const float mean = row_total(sum, red) / (float)width;
+        float m2 = 0.f;
+        for (int q = i0; q < nv; q += TPR) {
+            const float4 v = reinterpret_cast<const float4*>(xs)[q];
+            const float f[4] = {v.x - mean, v.y - mean, v.z - mean, v.w - mean};
 #pragma unroll
-            for (int w = 1; w < WPR; ++w) merge(p[3 * w], p[3 * w + 1], p[3 * w + 2]);
+            for (int j = 0; j < 4; ++j) m2 = 4 * q + j < width ? fmaf(f[j], f[j], m2) : m2;
         }
+        const float rstd = 1.0f / sqrtf(row_total(m2, red + LM_WARPS) / (float)width + eps);
+        if (WPR == 1) __syncthreads();     // the constants are in place
         if (!on) return;
-        const float rstd = 1.0f / sqrtf(m2 / (float)width + eps);
         bf16* X1 = X + (size_t)r * ld;
         bf16* X2 = X + (size_t)(RT + r) * ld;
-        auto put = [&](const float4& u, int q) {
-            const float f[4] = {u.x, u.y, u.z, u.w};
+        for (int q = i0; q < nv; q += TPR) {
+            const float4 v = reinterpret_cast<const float4*>(xs)[q];
+            const float f[4] = {v.x, v.y, v.z, v.w};
             float a[4], b[4];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int k = 4 * q + j;
-                const bool in = k < width;
                 const float d = (f[j] - mean) * rstd;
-                a[j] = in ? fmaf(d, __ldg(n1.w + k), __ldg(n1.b + k)) : 0.f;
-                b[j] = in && n2.w ? fmaf(d, __ldg(n2.w + k), __ldg(n2.b + k)) : 0.f;
+                const bool in = k < width;
+                a[j] = in ? fmaf(d, sc[k], sc[K + k]) : 0.f;
+                b[j] = in && n2.w ? fmaf(d, sc[2 * K + k], sc[3 * K + k]) : 0.f;
             }
             Store<bf16>::put2(X1 + 4 * q, a[0], a[1]);
             Store<bf16>::put2(X1 + 4 * q + 2, a[2], a[3]);
             Store<bf16>::put2(X2 + 4 * q, b[0], b[1]);
             Store<bf16>::put2(X2 + 4 * q + 2, b[2], b[3]);
-        };
-#pragma unroll
-        for (int i = 0; i < KEEP; ++i)
-            if (4 * (i0 + i * TPR) < K) put(v[i], i0 + i * TPR);
-        for (int q = i0 + KEEP * TPR; 4 * q < K; q += TPR)
-            put(q < nv ? __ldcg(reinterpret_cast<const float4*>(xr) + q) : make_float4(0.f, 0.f, 0.f, 0.f), q);
+        }
     }
     __device__ __forceinline__ int tile_of(int n) const { return n >= split ? 1 : 0; }
 };
@@ -598,47 +629,39 @@ struct StageLatentQ {
     }
     static constexpr int TILES = 1;
     static constexpr bool K_PARTS = false;
+    static __host__ __device__ size_t scratch(int RT, int K) { return (size_t)(RT + 1) * K * 4; }
+    __device__ __forceinline__ void constants(float* sc, int K) const {
+        for (int k = threadIdx.x; k < K; k += LM_THREADS) sc[k] = k < q_rank ? __ldg(norm_w + k) : 0.f;
+    }
     template <int RT>
-    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, int K, int M, int) const {
-        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, KEEP = 8;
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, float* sc, int K, int M, int) const {
+        constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, U = 4;
         const int r = threadIdx.x / TPR, i0 = threadIdx.x % TPR, warp = threadIdx.x >> 5;
         const bool on = r < M;
         const float* src = dq + (size_t)(on ? r : 0) * lddq;
-        float2 v[KEEP];
+        float* xs = sc + (size_t)(1 + r) * K;
         float ss = 0.f;
-        auto get = [&](int q) {   // elements 2q, 2q + 1 (lddq is even; past q_rank: zero)
-            float2 u = on && 2 * q < q_rank ? __ldcg(reinterpret_cast<const float2*>(src) + q) : make_float2(0.f, 0.f);
-            if (2 * q + 1 >= q_rank) u.y = 0.f;
-            return u;
-        };
+        for (int k0 = i0; k0 < K; k0 += U * TPR) {
+            float v[U];
 #pragma unroll
-        for (int i = 0; i < KEEP; ++i) {
-            v[i] = get(i0 + i * TPR);
-            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
-        }
-        for (int q = i0 + KEEP * TPR; 2 * q < q_rank; q += TPR) {
-            const float2 u = get(q);
-            ss = fmaf(u.x, u.x, fmaf(u.y, u.y, ss));
+            for (int u = 0; u < U; ++u) v[u] = k0 + u * TPR < q_rank ? __ldcg(src + k0 + u * TPR) : 0.f;
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+                if (k0 + u * TPR < K) {
+                    xs[k0 + u * TPR] = v[u];
+                    ss = fmaf(v[u], v[u], ss);
+                }
         }
         ss = warp_sum(ss);
-        if (WPR > 1) {
-            if ((threadIdx.x & 31) == 0) red[warp] = ss;
-            __syncthreads();
-            ss = 0.f;
+        if ((threadIdx.x & 31) == 0) red[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
 #pragma unroll
-            for (int w = 0; w < WPR; ++w) ss += red[r * WPR + w];
-        }
+        for (int w = 0; w < WPR; ++w) ss += red[r * WPR + w];
         if (!on) return;
         const float rinv = 1.0f / sqrtf(ss / (float)q_rank + eps);
-        bf16* Xr = X + (size_t)r * ld;
-        auto put = [&](const float2& u, int q) {
-            const float w0 = 2 * q < q_rank ? __ldg(norm_w + 2 * q) : 0.f, w1 = 2 * q + 1 < q_rank ? __ldg(norm_w + 2 * q + 1) : 0.f;
-            Store<bf16>::put2(Xr + 2 * q, u.x * rinv * w0, u.y * rinv * w1);
-        };
-#pragma unroll
-        for (int i = 0; i < KEEP; ++i)
-            if (2 * (i0 + i * TPR) < K) put(v[i], i0 + i * TPR);
-        for (int q = i0 + KEEP * TPR; 2 * q < K; q += TPR) put(get(q), q);
+        for (int k = 2 * i0; k < K; k += 2 * TPR)
+            Store<bf16>::put2(X + (size_t)r * ld + k, xs[k] * rinv * sc[k], xs[k + 1] * rinv * sc[k + 1]);
     }
     __device__ __forceinline__ int tile_of(int) const { return 0; }
 };
@@ -662,8 +685,10 @@ struct StageRowsT {
     __device__ __forceinline__ void extra(int) const {}
     static constexpr int TILES = 1;
     static constexpr bool K_PARTS = true;   // may stage one CTA's part of K alone
+    static __host__ __device__ size_t scratch(int, int) { return 0; }
+    __device__ __forceinline__ void constants(float*, int) const {}
     template <int RT>
-    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float*, int K, int M, int k0) const {
+    __device__ __forceinline__ void stage_rows(bf16* X, int ld, float*, float*, int K, int M, int k0) const {
         const int nv = K / 8;
         for (int r = 0; r < M; ++r)
             for (int v = threadIdx.x; v < nv; v += LM_THREADS)
@@ -683,8 +708,9 @@ struct StreamArgs {
 template <int RT, class Stage, class Epi>
 static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Epi ep, StreamArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    __shared__ float red[3 * LM_WARPS];
+    __shared__ float red[2 * LM_WARPS];
     __shared__ __align__(16) float part[LM_WARPS][16][8];
+    __shared__ float2 sums[LM_WARPS * 8 * 8];   // of the CTA's warps: pair of rows x activation row x group
     constexpr int U = 4;       // 32-k blocks per round, two rounds in flight
     bf16* X = reinterpret_cast<bf16*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
@@ -718,8 +744,19 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
     const int total = sets * rounds;
     load(0, 0, 0);
     if (total > 1) load(1, rounds > 1 ? 0 : 1, rounds > 1 ? 1 : 0);
+    {   // a few rounds more of the first set on their way to L2
+        const int grp = cta * gpc + gi;
+        if (grp < a.n_groups && t == 0)
+            for (int b = 2 * U; b < my_kb && b < 8 * U; ++b) {
+                const bf16* p = a.W + (size_t)(grp * 16 + g) * a.K + rank * Kc + (size_t)(kp + b * ksplit) * 32;
+                asm volatile("prefetch.global.L2 [%0];" ::"l"(p));
+                asm volatile("prefetch.global.L2 [%0];" ::"l"(p + (size_t)8 * a.K));
+            }
+    }
+    float* sc = reinterpret_cast<float*>(X + (size_t)Stage::TILES * RT * ld);
+    st.constants(sc, Kc);
     pdl_wait();
-    st.template stage_rows<RT>(X, ld, red, Kc, a.M, rank * Kc);
+    st.template stage_rows<RT>(X, ld, red, sc, Kc, a.M, rank * Kc);
     __syncthreads();
     const int xrow = min(g, a.M - 1);   // columns past the last row repeat it and are not stored
     int s = 0, it = 0;
@@ -758,41 +795,35 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
         // the set is complete: sums meet in shared memory
         *reinterpret_cast<float2*>(&part[warp][g][2 * t]) = make_float2(acc[0][0] + acc[1][0], acc[0][1] + acc[1][1]);
         *reinterpret_cast<float2*>(&part[warp][g + 8][2 * t]) = make_float2(acc[0][2] + acc[1][2], acc[0][3] + acc[1][3]);
-        if (a.ck > 1) {
-            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-        } else {
-            __syncthreads();
-        }
-        // 8 pairs of rows per group x M rows, dealt to the threads of the CTA (of the cluster)
-        const int base = (s * n_cta + cta) * gpc;
-        const int n_out = gpc * 8 * a.M;
-        for (int o = rank * LM_THREADS + threadIdx.x; o < n_out; o += a.ck * LM_THREADS) {
-            const int pr = o % 8, gm = o / 8, q = gm % gpc, m = gm / gpc;
-            if (base + q >= a.n_groups) continue;
+        __syncthreads();
+        // 8 pairs of rows x M rows x gpc groups: first over the CTA's warps, then over the cluster
+        const int base = (s * n_cta + cta) * gpc, n_out = gpc * 8 * a.M;
+        for (int o = threadIdx.x; o < n_out; o += LM_THREADS) {
+            const int pr = o & 7, gm = o >> 3, q = gm % gpc, m = gm / gpc;
             float v0 = 0.f, v1 = 0.f;
-            for (int c = 0; c < a.ck; ++c) {
-                for (int w = 0; w < a.kw; ++w) {
+#pragma unroll
+            for (int w = 0; w < LM_WARPS; ++w)
+                if (w < a.kw) {
                     const float* p = &part[q * a.kw + w][2 * pr][m];
-                    if (a.ck == 1) {
-                        v0 += p[0];
-                        v1 += p[8];
-                    } else {
-                        uint32_t ra;
-                        float f0, f1;
-                        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(p)), "r"(c));
-                        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(f0) : "r"(ra) : "memory");
-                        asm volatile("ld.shared::cluster.f32 %0, [%1 + 32];" : "=f"(f1) : "r"(ra) : "memory");
-                        v0 += f0;
-                        v1 += f1;
-                    }
+                    v0 += p[0];
+                    v1 += p[8];
                 }
-            }
-            ep.store(m, (base + q) * 16 + 2 * pr, v0, v1);
+            if (a.ck > 1) sums[o] = make_float2(v0, v1);
+            else if (base + q < a.n_groups) ep.store(m, (base + q) * 16 + 2 * pr, v0, v1);
         }
-        if (a.ck > 1) {   // no CTA leaves while a peer may still read its sums
-            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        if (a.ck > 1) {
+            cluster_arrive();
+            cluster_wait();
+            for (int o = rank + a.ck * threadIdx.x; o < n_out; o += a.ck * LM_THREADS) {
+                const int pr = o & 7, gm = o >> 3, q = gm % gpc, m = gm / gpc;
+                float2 v[4];
+#pragma unroll
+                for (int c = 0; c < 4; ++c) v[c] = c < a.ck ? ld_cluster2(cluster_addr(&sums[o], c)) : make_float2(0.f, 0.f);
+                if (base + q < a.n_groups)
+                    ep.store(m, (base + q) * 16 + 2 * pr, (v[0].x + v[1].x) + (v[2].x + v[3].x), (v[0].y + v[1].y) + (v[2].y + v[3].y));
+            }
+            cluster_arrive();   // no CTA leaves, or writes its sums again, while a peer may still read them
+            cluster_wait();
         } else if (s + 1 < sets) {
             __syncthreads();
         }
