@@ -18,7 +18,7 @@
 
 namespace vuib {
 
-constexpr int LA_KEYS = 64;        // keys per tile (bf16)
+constexpr int LA_KEYS = 128;       // most keys per tile (bf16): 16 per warp; wide rows take 64 or 32
 constexpr int LA_KEYS_F32 = 32;
 constexpr int LA_MAX_SPLITS = 64;
 
@@ -68,6 +68,7 @@ struct LatentAttnArgs {
     const int32_t* row_slot;
     const int32_t* row_pos;
     int H, Rp, Dp, max_seq, n_slots;
+    int keys;                 // per tile
     int nbuf;                 // key tiles in shared memory (1 or 2)
     float scale;
     FastDiv row_vecs, w_vecs; // Dp / 8, Rp / 8
@@ -76,7 +77,6 @@ struct LatentAttnArgs {
     const bf16* gate;         // (M, ldgate)
     bf16* out;                // fused: (M, ldo) gated values; else the latent sums
     int ldgate, ldo, vdim;
-    int w_smem;               // fused: the CTA's value matrices are brought to shared memory before the dependency wait
     // fp32: partial sums of the splits
     float* part;              // (M, S, H, Rp)
     float* ml;                // (M, S, H, 2): running maximum and sum
@@ -84,18 +84,19 @@ struct LatentAttnArgs {
     int col_blocks;           // grid.y = head groups of 16 x column blocks
 };
 
-// How the keys of a row of `len` positions are dealt to S splits in tiles of `keys`: tiles per split, splits in use.
-__device__ __forceinline__ void latent_splits(int len, int keys, int S, int& tps, int& ns) {
-    const int nt = (len + keys - 1) / keys;
-    tps = (nt + S - 1) / S;
-    ns = (nt + tps - 1) / tps;
+// How the keys of a row of `len` positions are dealt to S splits in units of `keys`: units per split, splits in use.
+__device__ __forceinline__ void latent_splits(int len, int keys, int S, int& ups, int& ns) {
+    const int nu = (len + keys - 1) / keys;
+    ups = (nu + S - 1) / S;
+    ns = (nu + ups - 1) / ups;
 }
+constexpr int LA_UNIT = 16;       // the bf16 kernel deals whole 16-key MMA steps
 
 constexpr int LA_MAX_CL = 8;      // CTAs (key splits) of a row's cluster
 
 // fuse_heads: heads a CTA finishes itself (0: it does not); w_rows: rows of the value matrices it keeps
-static inline size_t latent_attn_smem(int Dp, int Rp, int nbuf, int fuse_heads = 0, int w_rows = 0) {
-    const size_t keys = (size_t)nbuf * LA_KEYS * (Dp + 8) * 2, sums = (size_t)16 * (Rp + 4) * 4;   // share their space
+static inline size_t latent_attn_smem(int Dp, int Rp, int keys_per_tile, int nbuf, int fuse_heads = 0, int w_rows = 0) {
+    const size_t keys = (size_t)nbuf * keys_per_tile * (Dp + 8) * 2, sums = (size_t)16 * (Rp + 4) * 4;   // share their space
     return (size_t)16 * (Dp + 8) * 2 + (keys > sums ? keys : sums) + 16 * (LA_KEYS + 4) * 4 + 2 * 16 * (LA_KEYS + 8) * 2 +
            16 * 4 + 16 * 8 + (size_t)fuse_heads * Rp * 2 + (size_t)w_rows * (Rp + LS_PAD) * 2;
 }
@@ -112,7 +113,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);
     bf16* Ks = Qs + 16 * ld;
     float* Os = reinterpret_cast<float*>(Ks);          // [16][lds], once the keys are used up
-    const size_t ks_bytes = (size_t)a.nbuf * LA_KEYS * ld * 2, os_bytes = (size_t)16 * lds * 4;
+    const size_t ks_bytes = (size_t)a.nbuf * a.keys * ld * 2, os_bytes = (size_t)16 * lds * 4;
     float* Ss = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(Ks) + (ks_bytes > os_bytes ? ks_bytes : os_bytes));
     bf16* Ph = reinterpret_cast<bf16*>(Ss + 16 * SP);
     bf16* Pl = Ph + 16 * PP;
@@ -123,37 +124,42 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     const int hpc = 16 / CL, h_loc0 = sp * hpc, h0 = hg * 16 + h_loc0;   // heads this CTA finishes
     const int n_fin = max(0, min(hpc, a.H - h0));
     bf16* ol = reinterpret_cast<bf16*>(ml_s + 32);      // [hpc][Rp] merged sums (FUSE_V)
-    bf16* Ws = ol + (FUSE_V ? hpc * a.Rp : 0);          // [n_fin * vdim][Rp + LS_PAD] (FUSE_V, w_smem)
+    bf16* Ws = ol + (FUSE_V ? hpc * a.Rp : 0);          // [n_fin * vdim][Rp + LS_PAD] (FUSE_V)
     if constexpr (FUSE_V) {   // the value matrices are constants: on their way while the predecessor runs
         const bf16* p = a.wuv + (size_t)h0 * a.vdim * a.Rp;
         const int n = n_fin * a.vdim * a.Rp;            // a multiple of 16
-        if (a.w_smem) {
-            for (int i = tid; i < n / 8; i += LM_THREADS) cp_async16(Ws + i * 8 + a.w_vecs.div(i) * LS_PAD, p + i * 8, true);
-            cp_async_commit();
-        } else {
-            for (int i = tid * 64; i < n; i += LM_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + i));
-        }
+        for (int i = tid; i < n / 8; i += LM_THREADS) cp_async16(Ws + i * 8 + a.w_vecs.div(i) * LS_PAD, p + i * 8, true);
+        cp_async_commit();
         // The rows of this split, as the table reads now, on their way to L2: a hint only, read again below.
         const int s_ = min(max(__ldcg(a.row_slot + m), 0), a.n_slots - 1), l_ = min(max(__ldcg(a.row_pos + m), 0), a.max_seq - 1);
         int tps, ns;
-        latent_splits(l_ + 1, LA_KEYS, CL, tps, ns);
+        latent_splits(l_ + 1, LA_UNIT, CL, tps, ns);
         const bf16* kb = static_cast<const bf16*>(a.cache) + (size_t)s_ * a.max_seq * a.Dp;
-        const int e0 = min(l_, sp * tps * LA_KEYS) * a.Dp, e1 = min(l_, min((sp + 1) * tps, sp * tps + 4) * LA_KEYS) * a.Dp;
-        for (int i = e0 + tid * 64; i < e1; i += LM_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(kb + i));
+        const int e0 = min(l_, sp * tps * LA_UNIT) * a.Dp, e1 = min(l_, min((sp + 1) * tps * LA_UNIT, sp * tps * LA_UNIT + 2 * LA_KEYS)) * a.Dp;
+        for (int i = e0 + tid * 16; i < e1; i += LM_THREADS * 16) asm volatile("prefetch.global.L2 [%0];" ::"l"(kb + i));
     }
     pdl_wait();
     const int slot = __ldcg(a.row_slot + m), len = __ldcg(a.row_pos + m) + 1;
     int tps, ns;
-    latent_splits(len, LA_KEYS, CL, tps, ns);
-    const int k_begin = min(len, sp * tps * LA_KEYS), k_end = min(len, (sp + 1) * tps * LA_KEYS);
-    const int n_tiles = (k_end - k_begin + LA_KEYS - 1) / LA_KEYS;     // 0 for a split without keys
-    const int nv = a.Dp / 8;
+    latent_splits(len, LA_UNIT, CL, tps, ns);
+    const int k_begin = min(len, sp * tps * LA_UNIT), k_end = min(len, (sp + 1) * tps * LA_UNIT);
+    const int n_tiles = (k_end - k_begin + a.keys - 1) / a.keys;     // 0 for a split without keys
+    const int nv = a.Dp / 8, gph = (a.vdim + 15) / 16;
+    // gates of value rows group q (16 rows of a head): this lane's rows g and g + 8; the first group's are asked for now
+    auto gates = [&](int q, float& lo, float& hi) {
+        const int h = q / gph, d = (q - h * gph) * 16 + g;
+        const bf16* p = a.gate + (size_t)m * a.ldgate + (size_t)(h0 + h) * a.vdim + d;
+        lo = t == 0 && q < n_fin * gph && d < a.vdim ? bf2f(p[0]) : 0.f;
+        hi = t == 0 && q < n_fin * gph && d + 8 < a.vdim ? bf2f(p[8]) : 0.f;
+    };
+    float gate_lo = 0.f, gate_hi = 0.f;
+    if constexpr (FUSE_V) gates(warp, gate_lo, gate_hi);
     const bf16* kb = static_cast<const bf16*>(a.cache) + (size_t)slot * a.max_seq * a.Dp;
     auto fetch = [&](int tile) {   // a tile's rows are consecutive in memory
-        bf16* dst = Ks + (size_t)(tile % a.nbuf) * LA_KEYS * ld;
-        const int k0 = k_begin + tile * LA_KEYS, n = min(LA_KEYS, k_end - k0) * nv;
+        bf16* dst = Ks + (size_t)(tile % a.nbuf) * a.keys * ld;
+        const int k0 = k_begin + tile * a.keys, keys = min(a.keys, k_end - k0), n = keys * nv, n16 = (keys + 15) / 16 * 16 * nv;
         const bf16* src = kb + (size_t)k0 * a.Dp;
-        for (int i = tid; i < LA_KEYS * nv; i += LM_THREADS)
+        for (int i = tid; i < n16; i += LM_THREADS)      // zero rows up to the next MMA step
             cp_async16(dst + i * 8 + a.row_vecs.div(i) * 8, src + (i < n ? i : 0) * 8, i < n);
         cp_async_commit();
     };
@@ -177,51 +183,51 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
         if (ahead) cp_async_wait<1>();
         else cp_async_wait<0>();
         __syncthreads();
-        const bf16* K = Ks + (size_t)(tile % a.nbuf) * LA_KEYS * ld;
-        // ---- scores of 16 heads x 8 keys per warp, two independent accumulators
-        float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-        const bf16* qp = Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
-        const bf16* kp = K + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
-        int ks = 0;
+        const bf16* K = Ks + (size_t)(tile % a.nbuf) * a.keys * ld;
+        // ---- scores of 16 heads x 16 keys per warp
+        const int left = min(a.keys, k_end - k_begin - tile * a.keys);   // keys of this tile in range
+        const int key = warp * 16 + 2 * t;
+        if (warp * 16 < left) {
+            float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+            const bf16* qp = Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
+            const bf16* kp = K + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
 #pragma unroll 2
-        for (; ks + 2 <= ksteps; ks += 2) {
-            uint32_t a0[4], a1[4], b[4];
-            ldsm_x4(a0, qp + ks * 16);
-            ldsm_x4(a1, qp + ks * 16 + 16);
-            ldsm_x4(b, kp + ks * 16);
-            mma_bf16(s0, a0, b[0], b[1]);
-            mma_bf16(s1, a1, b[2], b[3]);
+            for (int ks = 0; ks < ksteps; ++ks) {
+                uint32_t q[4], b[4];
+                ldsm_x4(q, qp + ks * 16);
+                ldsm_x4(b, kp + ks * 16);      // keys +0..7 (k low, k high), keys +8..15
+                mma_bf16(s0, q, b[0], b[1]);
+                mma_bf16(s1, q, b[2], b[3]);
+            }
+            auto put = [&](int h, int k, float a0, float a1) {
+                *reinterpret_cast<float2*>(Ss + h * SP + k) = make_float2(k < left ? a0 * a.scale : NEG_BIG, k + 1 < left ? a1 * a.scale : NEG_BIG);
+            };
+            put(g, key, s0[0], s0[1]);
+            put(g + 8, key, s0[2], s0[3]);
+            put(g, key + 8, s1[0], s1[1]);
+            put(g + 8, key + 8, s1[2], s1[3]);
         }
-        if (ks < ksteps) {
-            uint32_t a0[4], b0, b1;
-            ldsm_x4(a0, qp + ks * 16);
-            ldsm_x2(b0, b1, K + (warp * 8 + (lane & 7)) * ld + ks * 16 + ((lane >> 3) & 1) * 8);
-            mma_bf16(s0, a0, b0, b1);
-        }
-        const int key = warp * 8 + 2 * t, left = k_end - k_begin - tile * LA_KEYS;   // keys of this tile in range
-        Ss[g * SP + key] = key < left ? (s0[0] + s1[0]) * a.scale : NEG_BIG;
-        Ss[g * SP + key + 1] = key + 1 < left ? (s0[1] + s1[1]) * a.scale : NEG_BIG;
-        Ss[(g + 8) * SP + key] = key < left ? (s0[2] + s1[2]) * a.scale : NEG_BIG;
-        Ss[(g + 8) * SP + key + 1] = key + 1 < left ? (s0[3] + s1[3]) * a.scale : NEG_BIG;
         __syncthreads();
-        // ---- softmax rows 2*warp, 2*warp + 1; lane holds keys 2*lane, 2*lane + 1
+        // ---- softmax rows 2*warp, 2*warp + 1; lane holds keys 4*lane .. 4*lane + 3
+        const bool has = 4 * lane < (left + 15) / 16 * 16;
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int h = 2 * warp + i;
-            const float2 v = *reinterpret_cast<const float2*>(Ss + h * SP + 2 * lane);
-            float mx = fmaxf(v.x, v.y);
+            const float4 v = has ? *reinterpret_cast<const float4*>(Ss + h * SP + 4 * lane) : make_float4(NEG_BIG, NEG_BIG, NEG_BIG, NEG_BIG);
+            float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             const float mn = fmaxf(m_run[i], mx);
             const float c = __expf(m_run[i] - mn);
-            const float p0 = v.x <= 0.5f * NEG_BIG ? 0.f : __expf(v.x - mn);
-            const float p1 = v.y <= 0.5f * NEG_BIG ? 0.f : __expf(v.y - mn);
-            l_run[i] = l_run[i] * c + warp_sum(p0 + p1);
+            auto weight = [&](float x) { return x <= 0.5f * NEG_BIG ? 0.f : __expf(x - mn); };
+            const float p0 = weight(v.x), p1 = weight(v.y), p2 = weight(v.z), p3 = weight(v.w);
+            l_run[i] = l_run[i] * c + warp_sum((p0 + p1) + (p2 + p3));
             m_run[i] = mn;
-            uint32_t hi, lo;
-            split_bf16x2(p0, p1, hi, lo);
-            *reinterpret_cast<uint32_t*>(Ph + h * PP + 2 * lane) = hi;
-            *reinterpret_cast<uint32_t*>(Pl + h * PP + 2 * lane) = lo;
+            uint32_t h0, l0, h1, l1;
+            split_bf16x2(p0, p1, h0, l0);
+            split_bf16x2(p2, p3, h1, l1);
+            *reinterpret_cast<uint2*>(Ph + h * PP + 4 * lane) = make_uint2(h0, h1);
+            *reinterpret_cast<uint2*>(Pl + h * PP + 4 * lane) = make_uint2(l0, l1);
             if (lane == 0) corr_s[h] = c;
         }
         __syncthreads();
@@ -232,8 +238,9 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
             acc[i][0] *= c_lo; acc[i][1] *= c_lo;
             acc[i][2] *= c_hi; acc[i][3] *= c_hi;
         }
-#pragma unroll 1
-        for (int j = 0; j < LA_KEYS / 16 && j * 16 < left; ++j) {
+#pragma unroll 2
+        for (int j = 0; j < LA_KEYS / 16; ++j) {
+            if (j * 16 >= left) break;
             uint32_t ph[4], pl[4];
             const int po = ((lane & 7) + ((lane >> 3) & 1) * 8) * PP + j * 16 + (lane >> 4) * 8;
             ldsm_x4(ph, Ph + po);
@@ -272,26 +279,39 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     // ---- merge: 256 / hpc threads per head
     const int tph = LM_THREADS / hpc, hl = tid / tph, c0 = tid % tph;
     if (hl < n_fin) {
-        float w[LA_MAX_CL], mx = NEG_BIG, l = 0.f;
+        constexpr int CB = 2;      // columns requested together
+        float w[LA_MAX_CL], o[CB][LA_MAX_CL], mx = NEG_BIG, l = 0.f;
         float2 p[LA_MAX_CL];
 #pragma unroll
-        for (int s = 0; s < LA_MAX_CL; ++s) {
+        for (int s = 0; s < LA_MAX_CL; ++s)
             p[s] = s < ns ? ld_cluster2(cluster_addr(ml_s + (h_loc0 + hl) * 2, s)) : make_float2(NEG_BIG, 0.f);
-            mx = fmaxf(mx, p[s].x);
-        }
+        auto ask = [&](int c) {
+#pragma unroll
+            for (int j = 0; j < CB; ++j)
+#pragma unroll
+                for (int s = 0; s < LA_MAX_CL; ++s)
+                    o[j][s] = s < ns && c + j * tph < a.Rp ? ld_cluster(cluster_addr(Os + (h_loc0 + hl) * lds + c + j * tph, s)) : 0.f;
+        };
+        ask(c0);
+#pragma unroll
+        for (int s = 0; s < LA_MAX_CL; ++s) mx = fmaxf(mx, p[s].x);
 #pragma unroll
         for (int s = 0; s < LA_MAX_CL; ++s) {
             w[s] = __expf(p[s].x - mx);
             l = fmaf(w[s], p[s].y, l);
         }
         const float inv = 1.0f / l;
-        for (int c = c0; c < a.Rp; c += tph) {
-            float o = 0.f;
+        for (int c = c0; c < a.Rp; c += CB * tph) {
+            if (c != c0) ask(c);
 #pragma unroll
-            for (int s = 0; s < LA_MAX_CL; ++s)
-                if (s < ns) o = fmaf(w[s], ld_cluster(cluster_addr(Os + (h_loc0 + hl) * lds + c, s)), o);
-            if constexpr (FUSE_V) ol[hl * a.Rp + c] = f2bf(o * inv);
-            else a.out[((size_t)m * a.H + h0 + hl) * a.Rp + c] = f2bf(o * inv);
+            for (int j = 0; j < CB; ++j) {
+                if (c + j * tph >= a.Rp) break;
+                float v = 0.f;
+#pragma unroll
+                for (int s = 0; s < LA_MAX_CL; ++s) v = fmaf(w[s], o[j][s], v);
+                if constexpr (FUSE_V) ol[hl * a.Rp + c + j * tph] = f2bf(v * inv);
+                else a.out[((size_t)m * a.H + h0 + hl) * a.Rp + c + j * tph] = f2bf(v * inv);
+            }
         }
     }
     __syncwarp();
@@ -299,21 +319,17 @@ static __global__ void __launch_bounds__(LM_THREADS) k_latent_attn(LatentAttnArg
     if constexpr (FUSE_V) {
         __syncthreads();
         // 16 value rows of a head per warp (the M side), k in the lanes' own order as in k_lm_stream; the N side is this row
-        const int gph = (a.vdim + 15) / 16, blocks = (a.Rp + 31) / 32, nkb = a.Rp / 32;
-        const size_t wst = a.w_smem ? a.Rp + LS_PAD : a.Rp;
-        const bf16* W = a.w_smem ? Ws : a.wuv + (size_t)h0 * a.vdim * a.Rp;
+        const int blocks = (a.Rp + 31) / 32, nkb = a.Rp / 32;
+        const int wst = a.Rp + LS_PAD;
         for (int q = warp; q < n_fin * gph; q += LM_WARPS) {
             const int h = q / gph, d0 = (q - h * gph) * 16;
             const int d_lo = d0 + g, d_hi = d0 + g + 8;
-            const bf16* w0 = W + ((size_t)h * a.vdim + min(d_lo, a.vdim - 1)) * wst + t * 8;
-            const bf16* w1 = W + ((size_t)h * a.vdim + min(d_hi, a.vdim - 1)) * wst + t * 8;
+            const bf16* w0 = Ws + (h * a.vdim + min(d_lo, a.vdim - 1)) * wst + t * 8;
+            const bf16* w1 = Ws + (h * a.vdim + min(d_hi, a.vdim - 1)) * wst + t * 8;
             const bf16* o = ol + h * a.Rp + t * 8;
             const size_t col = (size_t)(h0 + h) * a.vdim;
-            float g_lo = 0.f, g_hi = 0.f;
-            if (t == 0) {
-                if (d_lo < a.vdim) g_lo = bf2f(a.gate[(size_t)m * a.ldgate + col + d_lo]);
-                if (d_hi < a.vdim) g_hi = bf2f(a.gate[(size_t)m * a.ldgate + col + d_hi]);
-            }
+            float g_lo = gate_lo, g_hi = gate_hi;
+            if (q != warp) gates(q, g_lo, g_hi);
             float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4
             for (int b = 0; b < blocks; ++b) {

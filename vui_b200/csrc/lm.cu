@@ -361,7 +361,7 @@ LatentAttnArgs attn_args(VuibLm* e, int li) {
 template <bool FUSE_V>
 int32_t latent_attn_nt(VuibLm* e, const LatentAttnArgs& a, int CL, int M, cudaStream_t s) {
     const dim3 grid(CL * ((a.H + 15) / 16), M);
-    const size_t sm = latent_attn_smem(a.Dp, a.Rp, a.nbuf, FUSE_V ? 16 / CL : 0, FUSE_V && a.w_smem ? 16 / CL * a.vdim : 0);
+    const size_t sm = latent_attn_smem(a.Dp, a.Rp, a.keys, a.nbuf, FUSE_V ? 16 / CL : 0, FUSE_V ? 16 / CL * a.vdim : 0);
     if (a.Rp <= 128) return run_cl(e, k_latent_attn<2, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
     if (a.Rp <= 256) return run_cl(e, k_latent_attn<4, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
     if (a.Rp <= 512) return run_cl(e, k_latent_attn<8, FUSE_V>, grid, CL, LM_THREADS, sm, s, a, CL);
@@ -376,16 +376,19 @@ int32_t absorbed_attention_bf16(VuibLm* e, int li, int M, cudaStream_t s) {
     // splits of a row's keys: one wave of CTAs, no more than the cache has tiles
     const int units = M * ((l.heads + 15) / 16);
     int CL = 1;
-    while (CL < LA_MAX_CL && units * CL * 2 <= LA_CTAS && CL * LA_KEYS < e->cfg.max_seq) CL *= 2;
-    a.nbuf = latent_attn_smem(d.dp, d.rp, 2, 16) <= LM_MAX_SMEM ? 2 : 1;
+    while (CL < LA_MAX_CL && units * CL * 2 <= LA_CTAS && CL * LA_KEYS / 2 < e->cfg.max_seq) CL *= 2;
+    a.keys = LA_KEYS;
+    while (a.keys > 32 && latent_attn_smem(d.dp, d.rp, a.keys, 1) > LM_MAX_SMEM) a.keys /= 2;
+    const bool fuse = M <= LM_FEW_ROWS && latent_attn_smem(d.dp, d.rp, a.keys, 1, 16 / CL, 16 / CL * l.vdim) <= LM_MAX_SMEM;
+    // a second key tile in flight where it costs no resident CTA
+    a.nbuf = latent_attn_smem(d.dp, d.rp, a.keys, 2, fuse ? 16 / CL : 0, fuse ? 16 / CL * l.vdim : 0) <= (fuse ? LM_MAX_SMEM : LM_MAX_SMEM / 2) ? 2 : 1;
     a.wuv = static_cast<const bf16*>(e->w[li].w_uv);
     a.gate = wsp<bf16>(e, L.gate);
     a.ldgate = L.ld_gate;
     a.vdim = l.vdim;
     a.ldo = L.ld_ay;
-    if (M <= LM_FEW_ROWS) {
+    if (fuse) {
         a.out = wsp<bf16>(e, L.ay);
-        a.w_smem = latent_attn_smem(d.dp, d.rp, a.nbuf, 16 / CL, 16 / CL * l.vdim) <= 180 * 1024;
         return latent_attn_nt<true>(e, a, CL, M, s);
     }
     a.out = wsp<bf16>(e, L.olat);
@@ -658,7 +661,7 @@ extern "C" int32_t vuib_lm_create(const VuibLmConfig* cfg, const VuibLmLayer* la
             return VUIB_ERR_SHAPE;
         if (l.mlp != VUIB_LM_MLP_NONE && l.ff < 1) return VUIB_ERR_SHAPE;
         const VuibLmDims d = layer_dims(c, l);
-        if (c.dtype == VUIB_LM_BF16 ? d.rp > 1024 || latent_attn_smem(d.dp, d.rp, 1, 16) > LM_MAX_SMEM
+        if (c.dtype == VUIB_LM_BF16 ? d.rp > 1024 || latent_attn_smem(d.dp, d.rp, 32, 1) > LM_MAX_SMEM
                                     : latent_attn_f32_smem(d.dp) > LM_MAX_SMEM)
             return VUIB_ERR_SHAPE;
     }

@@ -300,6 +300,16 @@ static __global__ void __launch_bounds__(128) k_latent_rows(LatentRow a, const f
 // Pairwise epilogues: store(m, n, v0, v1) for the sums of weight rows n, n + 1 (n even) and activation row m.
 // ---------------------------------------------------------------------------
 
+// What an epilogue needs from global memory besides the sums may be asked for early: pre(m, n), then
+// store(m, n, v0, v1, pre).
+struct NoEpPre {};
+template <class Epi, class = void>
+struct EpPre {
+    typedef NoEpPre type;
+    static __device__ __forceinline__ type pre(const Epi&, int, int) { return NoEpPre{}; }
+    static __device__ __forceinline__ void store(const Epi& ep, int m, int n, float v0, float v1, const type&) { ep.store(m, n, v0, v1); }
+};
+
 // Everything a parallel block reads from x: [dq | dkv | gate] of the mixer, then the MLP's (gate, up) pairs.
 template <class T>
 struct EpBlockIn {
@@ -347,6 +357,10 @@ struct EpRotatedQ {
         const int j = n % head_rows - n0;
         put(m, n, j, v0, v1, j >= 0 && j < rot_dims ? trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) : nullptr);
     }
+    __device__ __forceinline__ float2 pre(int m, int n) const {
+        const int j = n % head_rows - n0;
+        return n < N && j >= 0 && j < rot_dims ? __ldg(trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) + (j >> 1)) : make_float2(1.f, 0.f);
+    }
     // tcgen05 form: the rows' (cos, sin) are fetched while the MMAs run, TC_EPI_BYTES_PER_M of them per row
     static constexpr int STAGE_DIMS = TC_EPI_BYTES_PER_M / 4;
     __device__ __forceinline__ void stage(unsigned char* es, int m_off, int M, int tid) const {
@@ -362,6 +376,17 @@ struct EpRotatedQ {
     __device__ __forceinline__ void store_staged(int m_off, int m, int n, float v0, float v1, const unsigned char* es) const {
         if (rot_dims > STAGE_DIMS) return store(m_off + m, n, v0, v1);
         if (n < N) put(m_off + m, n, n % head_rows - n0, v0, v1, reinterpret_cast<const float2*>(es) + m * (rot_dims / 2));
+    }
+};
+
+template <class T>
+struct EpPre<EpRotatedQ<T>> {
+    typedef float2 type;
+    static __device__ __forceinline__ float2 pre(const EpRotatedQ<T>& ep, int m, int n) { return ep.pre(m, n); }
+    static __device__ __forceinline__ void store(const EpRotatedQ<T>& ep, int m, int n, float v0, float v1, const float2& cs) {
+        if (n >= ep.N) return;
+        const float2 o = rotate_pair(v0, v1, cs);   // (1, 0) turns nothing
+        Store<T>::put2(ep.q + (size_t)m * ep.N + n, o.x, o.y);
     }
 };
 
@@ -746,9 +771,9 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
     if (total > 1) load(1, rounds > 1 ? 0 : 1, rounds > 1 ? 1 : 0);
     {   // a few rounds more of the first set on their way to L2
         const int grp = cta * gpc + gi;
-        if (grp < a.n_groups && t == 0)
+        if (grp < a.n_groups && (t & 1) == 0)     // a hint brings one 32-byte sector
             for (int b = 2 * U; b < my_kb && b < 8 * U; ++b) {
-                const bf16* p = a.W + (size_t)(grp * 16 + g) * a.K + rank * Kc + (size_t)(kp + b * ksplit) * 32;
+                const bf16* p = a.W + (size_t)(grp * 16 + g) * a.K + rank * Kc + (size_t)(kp + b * ksplit) * 32 + t * 8;
                 asm volatile("prefetch.global.L2 [%0];" ::"l"(p));
                 asm volatile("prefetch.global.L2 [%0];" ::"l"(p + (size_t)8 * a.K));
             }
@@ -756,6 +781,9 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
     float* sc = reinterpret_cast<float*>(X + (size_t)Stage::TILES * RT * ld);
     st.constants(sc, Kc);
     pdl_wait();
+    // of the output this thread stores first (below)
+    const int o_m = (threadIdx.x >> 3) / gpc, o_n = ((cta * gpc + (threadIdx.x >> 3) % gpc) * 16) + 2 * (threadIdx.x & 7);
+    const typename EpPre<Epi>::type first_pre = EpPre<Epi>::pre(ep, min(o_m, a.M - 1), o_n);
     st.template stage_rows<RT>(X, ld, red, sc, Kc, a.M, rank * Kc);
     __syncthreads();
     const int xrow = min(g, a.M - 1);   // columns past the last row repeat it and are not stored
@@ -809,7 +837,10 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
                     v1 += p[8];
                 }
             if (a.ck > 1) sums[o] = make_float2(v0, v1);
-            else if (base + q < a.n_groups) ep.store(m, (base + q) * 16 + 2 * pr, v0, v1);
+            else if (base + q < a.n_groups) {
+                const int n = (base + q) * 16 + 2 * pr;
+                EpPre<Epi>::store(ep, m, n, v0, v1, s == 0 && o < LM_THREADS ? first_pre : EpPre<Epi>::pre(ep, m, n));
+            }
         }
         if (a.ck > 1) {
             cluster_arrive();
