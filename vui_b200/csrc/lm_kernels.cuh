@@ -300,12 +300,13 @@ static __global__ void __launch_bounds__(128) k_latent_rows(LatentRow a, const f
 // Pairwise epilogues: store(m, n, v0, v1) for the sums of weight rows n, n + 1 (n even) and activation row m.
 // ---------------------------------------------------------------------------
 
-// What an epilogue needs from global memory besides the sums may be asked for early: pre(m, n), then
-// store(m, n, v0, v1, pre).
+// What an epilogue needs from global memory besides the sums may be asked for early, in two dependent steps around the
+// staging: ask(m), then pre(asked, n), then store(m, n, v0, v1, pre).
 struct NoEpPre {};
 template <class Epi, class = void>
 struct EpPre {
     typedef NoEpPre type;
+    static __device__ __forceinline__ int ask(const Epi&, int) { return 0; }
     static __device__ __forceinline__ type pre(const Epi&, int, int) { return NoEpPre{}; }
     static __device__ __forceinline__ void store(const Epi& ep, int m, int n, float v0, float v1, const type&) { ep.store(m, n, v0, v1); }
 };
@@ -357,9 +358,9 @@ struct EpRotatedQ {
         const int j = n % head_rows - n0;
         put(m, n, j, v0, v1, j >= 0 && j < rot_dims ? trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) : nullptr);
     }
-    __device__ __forceinline__ float2 pre(int m, int n) const {
+    __device__ __forceinline__ float2 turn(int pos, int n) const {
         const int j = n % head_rows - n0;
-        return n < N && j >= 0 && j < rot_dims ? __ldg(trig + (size_t)__ldcg(row_pos + m) * (rot_dims / 2) + (j >> 1)) : make_float2(1.f, 0.f);
+        return n < N && j >= 0 && j < rot_dims ? __ldg(trig + (size_t)pos * (rot_dims / 2) + (j >> 1)) : make_float2(1.f, 0.f);
     }
     // tcgen05 form: the rows' (cos, sin) are fetched while the MMAs run, TC_EPI_BYTES_PER_M of them per row
     static constexpr int STAGE_DIMS = TC_EPI_BYTES_PER_M / 4;
@@ -382,7 +383,8 @@ struct EpRotatedQ {
 template <class T>
 struct EpPre<EpRotatedQ<T>> {
     typedef float2 type;
-    static __device__ __forceinline__ float2 pre(const EpRotatedQ<T>& ep, int m, int n) { return ep.pre(m, n); }
+    static __device__ __forceinline__ int ask(const EpRotatedQ<T>& ep, int m) { return __ldcg(ep.row_pos + m); }
+    static __device__ __forceinline__ float2 pre(const EpRotatedQ<T>& ep, int asked, int n) { return ep.turn(asked, n); }
     static __device__ __forceinline__ void store(const EpRotatedQ<T>& ep, int m, int n, float v0, float v1, const float2& cs) {
         if (n >= ep.N) return;
         const float2 o = rotate_pair(v0, v1, cs);   // (1, 0) turns nothing
@@ -783,8 +785,9 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
     pdl_wait();
     // of the output this thread stores first (below)
     const int o_m = (threadIdx.x >> 3) / gpc, o_n = ((cta * gpc + (threadIdx.x >> 3) % gpc) * 16) + 2 * (threadIdx.x & 7);
-    const typename EpPre<Epi>::type first_pre = EpPre<Epi>::pre(ep, min(o_m, a.M - 1), o_n);
+    const int asked = EpPre<Epi>::ask(ep, min(o_m, a.M - 1));
     st.template stage_rows<RT>(X, ld, red, sc, Kc, a.M, rank * Kc);
+    const typename EpPre<Epi>::type first_pre = EpPre<Epi>::pre(ep, asked, o_n);
     __syncthreads();
     const int xrow = min(g, a.M - 1);   // columns past the last row repeat it and are not stored
     int s = 0, it = 0;
@@ -839,7 +842,7 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_lm_stream(Stage st, Ep
             if (a.ck > 1) sums[o] = make_float2(v0, v1);
             else if (base + q < a.n_groups) {
                 const int n = (base + q) * 16 + 2 * pr;
-                EpPre<Epi>::store(ep, m, n, v0, v1, s == 0 && o < LM_THREADS ? first_pre : EpPre<Epi>::pre(ep, m, n));
+                EpPre<Epi>::store(ep, m, n, v0, v1, s == 0 && o < LM_THREADS ? first_pre : EpPre<Epi>::pre(ep, EpPre<Epi>::ask(ep, m), n));
             }
         }
         if (a.ck > 1) {
