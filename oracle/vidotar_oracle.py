@@ -1,6 +1,6 @@
 """Plain CPU implementation of the Vidotar language model, one function per mechanism.
 
-TEST INFRASTRUCTURE ONLY: the checker of ``vui_b200``'s token-model path.  It shares no code with the product,
+TEST INFRASTRUCTURE ONLY: what the tests hold ``vui_b200``'s token-model path against.  It shares no code with the product,
 keeps no cache (every call attends over the whole sequence) and computes in the dtype of the weights it is given
 (float64 in the tests), so a difference from it is a difference of the product.
 
