@@ -14,7 +14,7 @@ from tests import token_models as tm
 from vui_b200 import TokenLM, Vidotar, VuiB200, _lib, load_model
 from vui_b200 import registry, trace
 from vui_b200.slots import SlotEngine
-from vui_b200.token_lm import abi_layer, pack_layer, trig_table
+from vui_b200.token_lm import abi_config, abi_layers, pack_layer, trig_table
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
@@ -29,12 +29,9 @@ def _save(folder, cfg, sd):
 
 def _handle(cfg, dtype=_lib.LM_BF16, **kw):
     c = Vidotar.parse_config(cfg)
-    a = dict(vocab=c.vocab, width=c.width, n_layers=len(c.layers), dtype=dtype, n_slots=3, max_seq=256, max_rows=2,
-             max_prefill_rows=64, norm_eps=c.norm_eps, embed_scale=c.embed_scale)
-    a.update(kw)
+    a = abi_config(c, **{**dict(dtype=dtype, n_slots=3, max_seq=256, max_rows=2, max_prefill_rows=64), **kw})
     h = C.c_void_p()
-    layers = (_lib.VuibLmLayer * len(c.layers))(*[abi_layer(s) for s in c.layers])
-    return _lib.load_lm().vuib_lm_create(C.byref(_lib.VuibLmConfig(**a)), layers, C.byref(h)), h
+    return _lib.load_lm().vuib_lm_create(C.byref(a), abi_layers(c), C.byref(h)), h
 
 
 def _dims(h, n):
@@ -184,12 +181,12 @@ def test_lm_symbols_match_the_header():
     names = sorted(set(re.findall(r"\b(vuib_lm_[a-z0-9_]+)\s*\(", src)))
     lib = _lib.load_lm()
     assert names == sorted(_lib.LM_SYMBOLS) and all(hasattr(lib, n) for n in names)
-    assert C.sizeof(_lib.VuibLmConfig) == 40 and C.sizeof(_lib.VuibLmLayer) == 56 and C.sizeof(_lib.VuibLmDims) == 80
+    assert C.sizeof(_lib.VuibLmConfig) == 48 and C.sizeof(_lib.VuibLmLayer) == 80 and C.sizeof(_lib.VuibLmDims) == 120
 
 
 def test_lm_create_validates_and_refuses_unbound_calls():
     lib, cfg = _lib.load_lm(), tm.CONFIGS["plain"]
-    assert _handle(cfg, dtype=7)[0] == -2 and _handle(cfg, max_seq=0)[0] == -3 and _handle(cfg, vocab=0)[0] == -2
+    assert _handle(cfg, dtype=7)[0] == -2 and _handle(cfg, max_seq=0)[0] == -3 and _handle({**cfg, "vocab": 0})[0] == -2
     c = json.loads(json.dumps(cfg))
     c["layers"][0]["mixer"]["rot"]["dims"] = 14   # more than the head has
     assert _handle(c)[0] == -2

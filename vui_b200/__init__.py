@@ -7,8 +7,8 @@ from .engine import Engine, GenConfig, RenderRequest, Row, Segment
 from .model import VuiB200, VuiShape
 from .registry import load_model, open_engine
 from .token_engine import TokenEngine, TokenGenConfig, TokenRow
-from .token_lm import TokenLM, Vidotar
+from .token_lm import Medirax, TokenLM, Vidotar
 
-__all__ = ["CodecCtx", "Engine", "GenConfig", "QwenCodecDecoder", "QwenCodecEncoder", "RenderRequest", "Row", "Segment",
+__all__ = ["CodecCtx", "Engine", "GenConfig", "Medirax", "QwenCodecDecoder", "QwenCodecEncoder", "RenderRequest", "Row", "Segment",
            "StreamingCodecEncoder", "TokenEngine", "TokenGenConfig", "TokenLM", "TokenRow", "Vidotar", "VuiB200", "VuiShape",
            "load_model", "open_engine"]

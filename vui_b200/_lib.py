@@ -26,7 +26,7 @@ UNITS = {
     "vuib200.cu": [*_COMMON, "fused_blocks.cuh", "depth_group.cuh", "prefill_attn.cuh"],
     "codec.cu": ["codec_kernels.cuh"],
     "codec_enc.cu": ["codec_enc_kernels.cuh"],
-    "lm.cu": [*_COMMON, "lm_kernels.cuh", "latent_attn.cuh", "latent_prefill.cuh"],
+    "lm.cu": [*_COMMON, "lm_kernels.cuh", "latent_attn.cuh", "latent_prefill.cuh", "grouped_attn.cuh", "delta_rule.cuh"],
 }
 # library -> (its units, the API headers they include)
 LIBRARIES = {
@@ -210,29 +210,34 @@ SYMBOLS = {
 }
 
 # ---------------------------------------------------------------------------- include/vuib200_lm.h
+LM_ABI_VERSION = 2
 LM_BF16, LM_F32 = 0, 1
-LM_MIX_LATENT = 1
-LM_MLP_NONE, LM_MLP_CLAMPED_GLU = 0, 1
+LM_MIX_LATENT, LM_MIX_GROUPED, LM_MIX_DELTA = 1, 2, 3
+LM_MLP_NONE, LM_MLP_CLAMPED_GLU, LM_MLP_RELU2 = 0, 1, 2
+LM_BLOCK_LN2, LM_BLOCK_RMS = 0, 1
 
 
 class VuibLmConfig(C.Structure):
-    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "n_layers", "dtype", "n_slots", "max_seq", "max_rows",
-                                         "max_prefill_rows")] + [("norm_eps", C.c_float), ("embed_scale", C.c_float)]
+    _fields_ = [(n, C.c_int32) for n in ("vocab", "width", "n_layers", "dtype", "block", "n_slots", "max_seq", "max_rows",
+                                         "max_prefill_rows")] + [(n, C.c_float) for n in ("norm_eps", "embed_scale", "logit_scale")]
 
 
 class VuibLmLayer(C.Structure):
-    _fields_ = [(n, C.c_int32) for n in ("mixer", "mlp", "heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank", "q_rank",
-                                         "ff")] + [(n, C.c_float) for n in ("scale", "mlp_limit", "mlp_slope", "mlp_shift")]
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "mlp", "heads", "kv_heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank",
+                                         "q_rank", "window", "qk_norm", "taps", "ff")] + [
+        (n, C.c_float) for n in ("scale", "softcap", "unit_eps", "mlp_limit", "mlp_slope", "mlp_shift")]
 
 
 class VuibLmDims(C.Structure):
-    _fields_ = [(n, C.c_int32) for n in ("k_in", "n_dq", "n_kv", "n_gate", "n_mlp", "n_in", "rp", "rotp", "dp", "k_q", "n_q",
-                                         "k_out", "off_y", "n_out", "x_ok", "dimp", "vdp", "n_xq", "k_kv", "n_xkv")]
+    _fields_ = [(n, C.c_int32) for n in ("k_in", "n_gate", "n_mlp", "n_in", "k_out", "off_y", "n_out", "n_dq", "n_kv", "rp", "rotp",
+                                         "dp", "k_q", "n_q", "x_ok", "n_xq", "k_kv", "n_xkv", "dimp", "vdp", "n_key", "n_value",
+                                         "n_ab", "n_raw", "cap", "reserved")] + [(n, C.c_int64) for n in ("off_v", "slot_bytes")]
 
 
 class VuibLmLayerWeights(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("norm1_w", "norm1_b", "norm2_w", "norm2_b", "q_norm", "kv_norm", "w_in", "w_q",
-                                          "w_uv", "w_out", "w_xq", "w_xkv", "trig")]
+    _fields_ = [(n, C.c_void_p) for n in ("norm1_w", "norm1_b", "norm2_w", "norm2_b", "q_norm", "kv_norm", "w_in", "w_q", "w_uv",
+                                          "w_out", "w_xq", "w_xkv", "trig", "b_in", "b_out", "conv", "neg_a", "dt_bias",
+                                          "head_norm")]
 
 
 class VuibLmHeadWeights(C.Structure):
@@ -348,7 +353,7 @@ def build_library(force: bool = False, verbose: bool = False, paths=None) -> str
 _loaded: dict[str, C.CDLL] = {}
 
 
-def _load(path: str, symbols: dict, version: str) -> C.CDLL:
+def _load(path: str, symbols: dict, version: str, want: int) -> C.CDLL:
     if path in _loaded:
         return _loaded[path]
     if _stale(path) and (shutil.which("nvcc") or os.path.exists("/usr/local/cuda/bin/nvcc")):
@@ -360,7 +365,7 @@ def _load(path: str, symbols: dict, version: str) -> C.CDLL:
         fn = getattr(lib, name)  # AttributeError if the export is missing
         fn.restype = res
         fn.argtypes = args
-    if getattr(lib, version)() != 1:
+    if getattr(lib, version)() != want:
         raise RuntimeError(f"{os.path.basename(path)}: ABI version mismatch")
     _loaded[path] = lib
     return lib
@@ -368,12 +373,12 @@ def _load(path: str, symbols: dict, version: str) -> C.CDLL:
 
 def load() -> C.CDLL:
     """Load libvuib200 (building it when the sources are newer) and type every symbol."""
-    return _load(LIB_PATH, SYMBOLS, "vuib_abi_version")
+    return _load(LIB_PATH, SYMBOLS, "vuib_abi_version", 1)
 
 
 def load_lm() -> C.CDLL:
     """The same for libvuib200_lm."""
-    return _load(LM_LIB_PATH, LM_SYMBOLS, "vuib_lm_abi_version")
+    return _load(LM_LIB_PATH, LM_SYMBOLS, "vuib_lm_abi_version", LM_ABI_VERSION)
 
 
 class VuibError(RuntimeError):

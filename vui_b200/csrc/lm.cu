@@ -1,13 +1,16 @@
 // libvuib200_lm: C ABI over the token-model kernels (see include/vuib200_lm.h).  The host side validates, lays out the
 // caller's workspace and enqueues kernels on the caller's stream; it never allocates device memory.
 //
-// A layer is four launches for up to LM_FEW_ROWS rows
-//   [norms + every projection of x] [queries, cache append] [attention, value matrix, gate] [output + MLP down, residual]
-// and seven for more: row norms, tcgen05 GEMM, latent rows, tcgen05 GEMM, attention, value matrix, tcgen05 GEMM.  A
-// prefill of many rows expands keys and values instead (latent_prefill.cuh).  32-bit models: fp32 products, and the
-// attention's splits merge in a launch of their own.
+// A layer starts with [norms + every projection of x] and ends with [output + MLP down, residual]: two weight-streaming
+// launches for up to LM_FEW_ROWS rows, a norm launch and two tcgen05 GEMMs for more.  Between them:
+//   latent    [queries, cache append] [attention, value matrix, gate] for few rows; latent rows, tcgen05 GEMM, attention,
+//             value matrix for more; a prefill of many rows expands keys and values instead (latent_prefill.cuh)
+//   grouped   one launch in a decode step; [rotation, norms, cache append] [attention] otherwise (grouped_attn.cuh)
+//   delta     one launch in a decode step; [convolution, unit norms, gates] [recurrence] [norm, gate] otherwise (delta_rule.cuh)
+// 32-bit models: fp32 products, and the latent attention's splits merge in a launch of their own.
 #include "../../include/vuib200_lm.h"
 
+#include <algorithm>
 #include <cstdarg>
 #include <cstdio>
 #include <cstring>
@@ -17,6 +20,8 @@
 #include <utility>
 #include <vector>
 
+#include "delta_rule.cuh"
+#include "grouped_attn.cuh"
 #include "host_common.cuh"
 #include "latent_attn.cuh"
 #include "latent_prefill.cuh"
@@ -38,11 +43,12 @@ constexpr int LM_EXPAND_MIN = 64;      // rows of a call from which a prefill ex
 constexpr size_t LM_MAX_SMEM = 227 * 1024;
 
 struct LmLayout {
-    size_t flag, ctl, row_slot, row_pos, segs, xsegs, tiles, x, xn, dq, cq, dkv, gate, q, ay, part, ml, olat;
+    size_t flag, ctl, row_slot, row_pos, row_ext, segs, xsegs, tiles, x, xn, dq, cq, dkv, gate, q, ay, part, ml, olat;
     size_t tc_partial, tc_counters, xkv, xc;
+    size_t raw, dx, dg, dout;   // grouped and delta layers: fp32 rows of the input product; delta: k_delta_rows, recurrence
     size_t draw_ctr, rep_counts, rep_hist, rep_head, rep_filled;
     size_t total;
-    int ldx, ld_dq, ld_dkv, ld_gate, ld_ay, ld_q;
+    int ldx, ld_dq, ld_dkv, ld_gate, ld_ay, ld_q, ld_raw;
     int x_rows;      // expanded rows the workspace holds
 };
 
@@ -66,6 +72,7 @@ struct VuibLm {
     LmLayout lay;
     bool have_w, have_cache, have_ws;
     int R;                 // rows of scratch
+    bool recurrent;        // some layer's state is carried from token to token
     int few_rows;          // rows up to which the streaming products run for this model's sizes
     int num_sms;
     unsigned spin_limit;
@@ -107,26 +114,49 @@ T* wsp(VuibLm* e, size_t off) { return reinterpret_cast<T*>(e->ws + off); }
 VuibLmDims layer_dims(const VuibLmConfig& c, const VuibLmLayer& l) {
     VuibLmDims d;
     memset(&d, 0, sizeof(d));
+    const bool mlp = l.mlp != VUIB_LM_MLP_NONE, b16 = c.dtype == VUIB_LM_BF16;
     d.k_in = up(c.width, 64);
-    d.rp = up(l.kv_rank, 16);
-    d.rotp = up(l.rot_dim, 16);
-    d.dp = d.rp + d.rotp;
-    d.n_dq = up(l.q_rank, 16);
-    d.n_kv = d.n_dq + d.dp;
-    d.n_gate = d.n_kv + up(l.heads * l.vdim, 16);
-    d.n_mlp = up(d.n_gate, 128);
-    d.n_in = d.n_mlp + (l.mlp == VUIB_LM_MLP_NONE ? 0 : up(2 * l.ff, 128));
-    d.k_q = up(l.q_rank, 64);
-    d.n_q = up(l.heads * d.dp, 128);
-    d.off_y = up(l.heads * l.vdim, 64);
-    d.k_out = d.off_y + (l.mlp == VUIB_LM_MLP_NONE ? 0 : up(l.ff, 64));
     d.n_out = up(c.width, 128);
     d.dimp = up(l.dim, 16);
     d.vdp = up(l.vdim, 16);
-    d.x_ok = c.dtype == VUIB_LM_BF16 && latent_prefill_fits(d.dimp + d.rotp, d.vdp);
-    d.n_xq = up(l.heads * (d.dimp + d.rotp), 128);
-    d.k_kv = up(d.rp, 64);
-    d.n_xkv = up(l.heads * (d.dimp + d.vdp), 128);
+    if (l.mixer == VUIB_LM_MIX_LATENT) {
+        d.rp = up(l.kv_rank, 16);
+        d.rotp = up(l.rot_dim, 16);
+        d.dp = d.rp + d.rotp;
+        d.n_dq = up(l.q_rank, 16);
+        d.n_kv = d.n_dq + d.dp;
+        d.n_gate = d.n_kv + up(l.heads * l.vdim, 16);
+        d.n_mlp = up(d.n_gate, 128);
+        d.k_q = up(l.q_rank, 64);
+        d.n_q = up(l.heads * d.dp, 128);
+        d.off_y = up(l.heads * l.vdim, 64);
+        d.x_ok = b16 && latent_prefill_fits(d.dimp + d.rotp, d.vdp);
+        d.n_xq = up(l.heads * (d.dimp + d.rotp), 128);
+        d.k_kv = up(d.rp, 64);
+        d.n_xkv = up(l.heads * (d.dimp + d.vdp), 128);
+        d.slot_bytes = (int64_t)c.max_seq * d.dp * (b16 ? 2 : 4);
+    } else {
+        const bool delta = l.mixer == VUIB_LM_MIX_DELTA;
+        d.n_key = (delta ? l.kv_heads : l.heads) * d.dimp;
+        d.n_value = d.n_key + l.kv_heads * d.dimp;
+        d.n_ab = d.n_value + (delta ? l.heads : l.kv_heads) * d.vdp;
+        d.n_raw = d.n_ab + (delta ? up(2 * l.heads, 16) : 0);
+        d.n_gate = d.n_raw + (delta ? l.heads * d.vdp : 0);
+        d.n_mlp = d.n_gate;
+        d.off_y = up(l.heads * d.vdp, 64);
+        if (delta) {
+            d.off_v = (int64_t)l.heads * d.vdp * d.dimp;
+            d.slot_bytes = 4 * (d.off_v + (int64_t)l.taps * d.n_ab);
+        } else {
+            // the ring: a window (read from a multiple of LA_UNIT on) and the rows of one call, or every position
+            const int64_t all = up(c.max_seq, GP_TILE), part = l.window > 0 ? ((int64_t)l.window + LA_UNIT + c.max_prefill_rows + GP_TILE - 1) / GP_TILE * GP_TILE : all;
+            d.cap = (int32_t)(part < all ? part : all);
+            d.off_v = (int64_t)l.kv_heads * d.cap * d.dimp;
+            d.slot_bytes = (d.off_v + (int64_t)l.kv_heads * d.cap * d.vdp) * (b16 ? 2 : 4);
+        }
+    }
+    d.n_in = up(d.n_mlp + (mlp ? (l.mlp == VUIB_LM_MLP_CLAMPED_GLU ? 2 : 1) * l.ff : 0), 128);
+    d.k_out = d.off_y + (mlp ? up(l.ff, 64) : 0);
     return d;
 }
 
@@ -147,12 +177,25 @@ void make_layout(VuibLm* e) {
     const size_t R = e->R, es = c.dtype == VUIB_LM_BF16 ? 2 : 4;
     size_t off = 0;
     auto take = [&](size_t bytes) { size_t o = off; off = align_up(off + bytes); return o; };
-    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0, olat = 0;
+    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0, olat = 0, raw = 0, dx = 0, dg = 0, dout = 0;
     size_t part = 0, ml = 0;
     for (size_t i = 0; i < e->layer.size(); ++i) {
         const VuibLmLayer& l = e->layer[i];
         const VuibLmDims& d = e->dims[i];
         auto mx = [](int& a, int b) { if (b > a) a = b; };
+        mx(ay, d.k_out);
+        if (l.mixer != VUIB_LM_MIX_LATENT) {
+            mx(raw, d.n_raw);
+            mx(gate, d.n_gate - d.n_raw);
+            if (l.mixer == VUIB_LM_MIX_GROUPED) {
+                mx(q, l.heads * d.dimp);
+            } else {
+                mx(dx, d.n_ab);
+                mx(dg, 2 * l.heads);
+                mx(dout, l.heads * d.vdp);
+            }
+            continue;
+        }
         mx(dq, d.n_dq);
         mx(cq, d.k_q);
         mx(dkv, d.dp);
@@ -163,7 +206,6 @@ void make_layout(VuibLm* e) {
             mx(xkv, l.heads * (d.dimp + d.vdp));
             mx(xc, d.k_kv);
         }
-        mx(ay, d.k_out);
         mx(olat, l.heads * d.rp);
         for (int m = 1; c.dtype == VUIB_LM_F32 && m <= LA_ROW_BLOCK && m <= (int)R; ++m) {
             const size_t rows = (size_t)m * attn_splits(e, (int)i, m) * l.heads;
@@ -177,11 +219,13 @@ void make_layout(VuibLm* e) {
     L.ld_gate = gate;
     L.ld_ay = ay;
     L.ld_q = q;
+    L.ld_raw = raw;
     L.x_rows = xkv ? (int)R + c.max_seq : 0;
     L.flag = take(256);
     L.ctl = take(sizeof(SamplingCtl));
     L.row_slot = take(R * 4);
     L.row_pos = take(R * 4);
+    L.row_ext = take(R * 8);
     L.segs = take(R * 16);
     L.xsegs = take(R * 16);
     L.tiles = take(R * 32);
@@ -200,6 +244,10 @@ void make_layout(VuibLm* e) {
     L.tc_counters = take(2 * TC_COUNTERS * 4);
     L.xkv = take((size_t)L.x_rows * xkv * es);
     L.xc = take((size_t)L.x_rows * xc * es);
+    L.raw = take(R * raw * 4);
+    L.dx = take(R * dx * 4);
+    L.dg = take(R * dg * 4);
+    L.dout = take(R * dout * 4);
     L.draw_ctr = take((size_t)c.n_slots * 4);
     L.rep_counts = take((size_t)c.n_slots * c.vocab * 4);
     L.rep_hist = take((size_t)c.n_slots * REP_HIST_MAX * 4);
@@ -302,15 +350,20 @@ int few_rows_of(const VuibLm* e) {
     const bool b16 = c.dtype == VUIB_LM_BF16;
     for (int rt = b16 ? LM_FEW_ROWS : LM_FEW_ROWS_F32; rt >= 1; rt /= 2) {
         bool ok = true;
-        for (const VuibLmDims& d : e->dims) {
+        for (size_t i = 0; i < e->dims.size(); ++i) {
+            const VuibLmDims& d = e->dims[i];
+            const bool latent = e->layer[i].mixer == VUIB_LM_MIX_LATENT;
+            size_t most;
             if (b16) {
-                ok = ok && stream_smem<StageLayerNorm2<bf16>>(rt, d.k_in, 1) <= LS_MAX_SMEM &&
-                     stream_smem<StageLatentQ<bf16>>(rt, d.k_q, 1) <= LS_MAX_SMEM &&
-                     stream_smem<StageRowsT<bf16>>(rt, d.k_out, stream_ck(up(c.width, 16) / 16, d.k_out, true)) <= LS_MAX_SMEM;
+                most = stream_smem<StageRowsT<bf16>>(rt, d.k_out, stream_ck(up(c.width, 16) / 16, d.k_out, true));
+                const size_t in = latent ? stream_smem<StageLayerNorm2<bf16>>(rt, d.k_in, 1) : stream_smem<StageRms<bf16>>(rt, d.k_in, 1);
+                const size_t q = latent ? stream_smem<StageLatentQ<bf16>>(rt, d.k_q, 1) : 0;
+                most = std::max(most, std::max(in, q));
             } else {   // one row at a time will do
-                ok = ok && StageLayerNorm2<float>::smem(1, d.k_in) <= LS_MAX_SMEM && StageRowsT<float>::smem(1, d.k_out) <= LS_MAX_SMEM &&
-                     StageRowsT<float>::smem(1, d.k_q) <= LS_MAX_SMEM;
+                most = std::max(StageRowsT<float>::smem(1, d.k_out), StageRowsT<float>::smem(1, d.k_q));
+                most = std::max(most, latent ? StageLayerNorm2<float>::smem(1, d.k_in) : StageRms<float>::smem(1, d.k_in));
             }
+            ok = ok && most <= LS_MAX_SMEM;
         }
         if (ok) return rt;
     }
@@ -498,75 +551,247 @@ int32_t expanded_attention(VuibLm* e, int li, const ExpandGroup& g, cudaStream_t
 }
 
 // ---------------------------------------------------------------------------
-// One pass over the layers for M rows whose x, slots and positions are in the workspace.
+// What a pass over the layers knows of its rows besides what is in the workspace.
 // ---------------------------------------------------------------------------
-template <class T>
-int32_t run_layers(VuibLm* e, int M, const std::vector<ExpandGroup>* expand, cudaStream_t s) {
+struct Pass {
+    int M;
+    bool step;         // a decode step: every row one token of a slot of its own
+    int n_segs;        // portions of a prefill
+    int n_tiles;       // query tiles of a prefill that runs the mixers' prefill forms (0: it does not)
+    const std::vector<ExpandGroup>* expand;
+    bool few;          // the weight-streaming products run
+};
+
+// The input product of a layer: norm (few rows: in the staging) and every matrix that reads x.
+template <class T, class Stage, class Epi>
+int32_t product_in(VuibLm* e, int li, const Pass& ps, const Stage& st, const Epi& ep, NormVec n1, NormVec n2, int n_split, cudaStream_t s) {
     const VuibLmConfig& c = e->cfg;
     const LmLayout& L = e->lay;
+    const VuibLmDims& d = e->dims[li];
+    if (ps.few) return few<T>(e, st, ep, e->w[li].w_in, d.k_in, ps.M, d.n_in, s);
+    T* xn = wsp<T>(e, L.xn);
+    T* xn2 = n2.w ? xn + (size_t)e->R * L.ldx : nullptr;
+    auto norm = c.block == VUIB_LM_BLOCK_LN2 ? k_norm_rows<T, true> : k_norm_rows<T, false>;
+    RC(run(e, norm, dim3(ps.M), 128, 0, s, wsp<float>(e, L.x), L.ldx, c.width, c.norm_eps, n1, xn, n2, xn2, L.ldx, nullptr, nullptr,
+           nullptr, nullptr));
+    return gemm<T>(e, e->maps[li].w_in, e->w[li].w_in, xn, L.ldx, d.k_in, ps.M, d.n_in, ep, s, n_split, e->R);
+}
+
+// x += W_out [mixer | MLP] (+ bias)
+template <class T>
+int32_t product_out(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
+    const LmLayout& L = e->lay;
+    const VuibLmDims& d = e->dims[li];
+    const T* ay = wsp<T>(e, L.ay);
+    const EpAddResidual er{wsp<float>(e, L.x), L.ldx, e->cfg.width, e->w[li].b_out};
+    if (ps.few) return few<T>(e, StageRowsT<T>{ay, L.ld_ay}, er, e->w[li].w_out, d.k_out, ps.M, e->cfg.width, s);
+    return gemm<T>(e, e->maps[li].w_out, e->w[li].w_out, ay, L.ld_ay, d.k_out, ps.M, d.n_out, er, s);
+}
+
+template <class T>
+int32_t latent_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
+    const VuibLmConfig& c = e->cfg;
+    const LmLayout& L = e->lay;
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    const VuibLmLayerWeights& w = e->w[li];
+    const LmMaps& mp = e->maps[li];
+    const int M = ps.M;
     float* x = wsp<float>(e, L.x);
-    const bool stream = M <= e->few_rows;
-    for (int li = 0; li < c.n_layers; ++li) {
-        const VuibLmLayer& l = e->layer[li];
-        const VuibLmDims& d = e->dims[li];
-        const VuibLmLayerWeights& w = e->w[li];
-        const LmMaps& mp = e->maps[li];
-        const bool ex = expand && d.x_ok && !stream;
-        const LayerNormW n1{w.norm1_w, w.norm1_b}, n2{w.norm2_w, w.norm2_b};
-        const float2* trig = reinterpret_cast<const float2*>(w.trig);
-        T* ay = wsp<T>(e, L.ay);
-        EpBlockIn<T> ei;
-        ei.n_dq = d.n_dq;
-        ei.n_kv = d.n_kv;
-        ei.n_gate = d.n_gate;
-        ei.n_mlp = d.n_mlp;
-        ei.ff = l.mlp == VUIB_LM_MLP_NONE ? 0 : l.ff;
-        ei.dq = wsp<float>(e, L.dq);
-        ei.lddq = L.ld_dq;
-        ei.dkv = wsp<float>(e, L.dkv);
-        ei.lddkv = d.dp;
-        ei.gate = wsp<T>(e, L.gate);
-        ei.ldgate = L.ld_gate;
-        ei.act = ay + d.off_y;
-        ei.ldact = L.ld_ay;
-        ei.limit = l.mlp_limit;
-        ei.slope = l.mlp_slope;
-        ei.shift = l.mlp_shift;
-        const LatentRow lat{wsp<float>(e, L.dkv), w.kv_norm, c.norm_eps, l.kv_rank, d.rp, l.rot_dim, l.rot_dims, d.dp, trig,
-                            e->cache[li], wsp<int32_t>(e, L.row_slot), wsp<int32_t>(e, L.row_pos), c.max_seq};
-        const int head_rows = ex ? d.dimp + d.rotp : d.dp;
-        const EpRotatedQ<T> eq{wsp<T>(e, L.q), l.heads * head_rows, head_rows, head_rows - d.rotp, l.rot_dims, trig,
-                               wsp<int32_t>(e, L.row_pos)};
-        const EpAddResidual er{x, L.ldx, c.width};
-        if (stream) {
-            const StageLayerNorm2<T> sn{x, L.ldx, c.width, c.norm_eps, n1, n2, d.n_mlp, nullptr};
-            RC(few<T>(e, sn, ei, w.w_in, d.k_in, M, d.n_in, s));
-            const StageLatentQ<T> sq{wsp<float>(e, L.dq), L.ld_dq, l.q_rank, c.norm_eps, w.q_norm, lat};
-            RC(few<T>(e, sq, eq, w.w_q, d.k_q, M, l.heads * d.dp, s));
-            RC(absorbed_attention<T>(e, li, M, s));
-            const StageRowsT<T> sr{ay, L.ld_ay};
-            RC(few<T>(e, sr, er, w.w_out, d.k_out, M, c.width, s));
+    const bool ex = ps.expand && d.x_ok && !ps.few;
+    const NormVec n1{w.norm1_w, w.norm1_b}, n2{w.norm2_w, w.norm2_b};
+    const float2* trig = reinterpret_cast<const float2*>(w.trig);
+    EpBlockIn<T> ei;
+    ei.n_dq = d.n_dq;
+    ei.n_kv = d.n_kv;
+    ei.n_gate = d.n_gate;
+    ei.n_mlp = d.n_mlp;
+    ei.ff = l.mlp == VUIB_LM_MLP_NONE ? 0 : l.ff;
+    ei.dq = wsp<float>(e, L.dq);
+    ei.lddq = L.ld_dq;
+    ei.dkv = wsp<float>(e, L.dkv);
+    ei.lddkv = d.dp;
+    ei.gate = wsp<T>(e, L.gate);
+    ei.ldgate = L.ld_gate;
+    ei.act = wsp<T>(e, L.ay) + d.off_y;
+    ei.ldact = L.ld_ay;
+    ei.limit = l.mlp_limit;
+    ei.slope = l.mlp_slope;
+    ei.shift = l.mlp_shift;
+    const LatentRow lat{wsp<float>(e, L.dkv), w.kv_norm, c.norm_eps, l.kv_rank, d.rp, l.rot_dim, l.rot_dims, d.dp, trig,
+                        e->cache[li], wsp<int32_t>(e, L.row_slot), wsp<int32_t>(e, L.row_pos), c.max_seq};
+    const int head_rows = ex ? d.dimp + d.rotp : d.dp;
+    const EpRotatedQ<T> eq{wsp<T>(e, L.q), l.heads * head_rows, head_rows, head_rows - d.rotp, l.rot_dims, trig,
+                           wsp<int32_t>(e, L.row_pos)};
+    const StageLayerNorm2<T> sn{x, L.ldx, c.width, c.norm_eps, n1, n2, d.n_mlp, nullptr};
+    RC(product_in<T>(e, li, ps, sn, ei, n1, n2, d.n_mlp, s));
+    if (ps.few) {
+        const StageLatentQ<T> sq{{wsp<float>(e, L.dq), L.ld_dq, l.q_rank, c.norm_eps, w.q_norm}, lat};
+        RC(few<T>(e, sq, eq, w.w_q, d.k_q, M, l.heads * d.dp, s));
+    } else {
+        RC(run(e, k_latent_rows<T>, dim3(M), 128, 0, s, lat, wsp<float>(e, L.dq), L.ld_dq, l.q_rank, w.q_norm,
+               wsp<T>(e, L.cq), d.k_q));
+        RC(gemm<T>(e, ex ? mp.w_xq : mp.w_q, ex ? w.w_xq : w.w_q, wsp<T>(e, L.cq), d.k_q, d.k_q, M, ex ? d.n_xq : d.n_q, eq, s));
+    }
+    if (ex) {
+        if constexpr (std::is_same<T, bf16>::value) {
+            for (const ExpandGroup& g : *ps.expand) RC(expanded_attention(e, li, g, s));
+        }
+    } else {
+        RC(absorbed_attention<T>(e, li, M, s));
+    }
+    return product_out<T>(e, li, ps, s);
+}
+
+// The input product of the layers with one RMS norm.
+template <class T>
+int32_t mix_in(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
+    const VuibLmConfig& c = e->cfg;
+    const LmLayout& L = e->lay;
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    const NormVec n1{e->w[li].norm1_w, nullptr};
+    const EpMixIn<T> ei{d.n_raw, d.n_gate, d.n_mlp, l.mlp == VUIB_LM_MLP_NONE ? 0 : l.ff, e->w[li].b_in, wsp<float>(e, L.raw), L.ld_raw,
+                        wsp<T>(e, L.gate), L.ld_gate, wsp<T>(e, L.ay) + d.off_y, L.ld_ay};
+    const StageRms<T> st{wsp<float>(e, L.x), L.ldx, c.width, c.norm_eps, n1.w};
+    return product_in<T>(e, li, ps, st, ei, n1, NormVec{nullptr, nullptr}, 1 << 30, s);
+}
+
+template <bool OWN>
+int32_t grouped_rows_bf16(VuibLm* e, int li, const QkRowsArgs& r, int M, cudaStream_t s) {
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    GroupedAttnArgs a;
+    memset(&a, 0, sizeof(a));
+    a.r = r;
+    a.q = static_cast<const bf16*>(r.q);
+    a.out = wsp<bf16>(e, e->lay.ay);
+    a.ldo = e->lay.ld_ay;
+    a.window = l.window > 0 ? l.window : e->cfg.max_seq;
+    a.max_seq = e->cfg.max_seq;
+    a.n_slots = e->cfg.n_slots;
+    a.hpg = l.heads / l.kv_heads;
+    a.hgroups = (a.hpg + 15) / 16;
+    a.scale = l.scale;
+    a.softcap = l.softcap;
+    a.k_vecs = FastDiv(d.dimp / 8);
+    a.v_vecs = FastDiv(d.vdp / 8);
+    const int units = M * l.kv_heads * a.hgroups, seen = std::min(a.window, a.max_seq);
+    int CL = 1;
+    while (CL < LA_MAX_CL && units * CL * 2 <= LA_CTAS && CL * LA_KEYS / 2 < seen) CL *= 2;
+    a.keys = LA_KEYS;
+    while (a.keys > 32 && (grouped_attn_smem(d.dimp, d.vdp, a.keys, 1) > LM_MAX_SMEM || a.keys / 2 * CL >= seen + 16)) a.keys /= 2;
+    // a second key tile in flight where a split has more than one and it costs no resident CTA
+    a.nbuf = a.keys * CL < seen + 16 && grouped_attn_smem(d.dimp, d.vdp, a.keys, 2) <= LM_MAX_SMEM / 2 ? 2 : 1;
+    const dim3 grid(CL * a.hgroups * l.kv_heads, M);
+    const size_t sm = grouped_attn_smem(d.dimp, d.vdp, a.keys, a.nbuf);
+    if (d.vdp <= 128) return run_cl(e, k_grouped_attn<2, OWN>, grid, CL, LM_THREADS, sm, s, a, CL);
+    return run_cl(e, k_grouped_attn<4, OWN>, grid, CL, LM_THREADS, sm, s, a, CL);
+}
+
+template <int KS>
+int32_t grouped_tiles(VuibLm* e, const GroupedPrefillArgs& a, int n_tiles, cudaStream_t s) {
+    const dim3 grid(n_tiles, a.H);
+    const size_t sm = grouped_prefill_smem(a.c.dimp, a.c.vdp);
+    if (a.c.vdp <= 64) return run(e, k_grouped_prefill<KS, 4>, grid, 128, sm, s, a);
+    if (a.c.vdp <= 128) return run(e, k_grouped_prefill<KS, 8>, grid, 128, sm, s, a);
+    return run(e, k_grouped_prefill<KS, 16>, grid, 128, sm, s, a);
+}
+
+template <class T>
+int32_t grouped_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
+    const VuibLmConfig& c = e->cfg;
+    const LmLayout& L = e->lay;
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    RC(mix_in<T>(e, li, ps, s));
+    QkRowsArgs r;
+    memset(&r, 0, sizeof(r));
+    r.raw = wsp<float>(e, L.raw);
+    r.ldraw = L.ld_raw;
+    r.n_k = d.n_key;
+    r.n_v = d.n_value;
+    r.q = wsp<T>(e, L.q);
+    r.c = GroupedCache{e->cache[li], (size_t)d.slot_bytes / sizeof(T), (size_t)d.off_v, d.cap, d.dimp, d.vdp};
+    r.h = QkHead{reinterpret_cast<const float2*>(e->w[li].trig), l.dim, d.dimp, l.rot_dims, c.norm_eps, l.qk_norm};
+    r.row_slot = wsp<int32_t>(e, L.row_slot);
+    r.row_pos = wsp<int32_t>(e, L.row_pos);
+    r.H = l.heads;
+    r.G = l.kv_heads;
+    const int window = l.window > 0 ? l.window : c.max_seq, hpg = l.heads / l.kv_heads;
+    if constexpr (std::is_same<T, bf16>::value) {
+        if (ps.step) {
+            RC(grouped_rows_bf16<true>(e, li, r, ps.M, s));
         } else {
-            T* xn = wsp<T>(e, L.xn);
-            T* xn2 = xn + (size_t)e->R * L.ldx;
-            RC(run(e, k_layernorm_rows<T>, dim3(M), 128, 0, s, x, L.ldx, c.width, c.norm_eps, n1, xn, n2, w.norm2_w ? xn2 : nullptr,
-                   L.ldx, nullptr, nullptr, nullptr, nullptr));
-            RC(gemm<T>(e, mp.w_in, w.w_in, xn, L.ldx, d.k_in, M, d.n_in, ei, s, d.n_mlp, e->R));
-            RC(run(e, k_latent_rows<T>, dim3(M), 128, 0, s, lat, wsp<float>(e, L.dq), L.ld_dq, l.q_rank, w.q_norm,
-                   wsp<T>(e, L.cq), d.k_q));
-            RC(gemm<T>(e, ex ? mp.w_xq : mp.w_q, ex ? w.w_xq : w.w_q, wsp<T>(e, L.cq), d.k_q, d.k_q, M, ex ? d.n_xq : d.n_q, eq, s));
-            if (ex) {
-                if constexpr (std::is_same<T, bf16>::value) {
-                    for (const ExpandGroup& g : *expand) RC(expanded_attention(e, li, g, s));
-                }
+            RC(run(e, k_qk_rows<T>, dim3(ps.M), LM_THREADS, 0, s, r));
+            if (ps.n_tiles) {
+                const GroupedPrefillArgs a{static_cast<const bf16*>(r.q), r.c, wsp<int4>(e, L.tiles), wsp<bf16>(e, L.ay), L.ld_ay, l.heads,
+                                           hpg, window, l.scale, l.softcap, FastDiv((d.dimp + d.vdp) / 8)};
+                if (d.dimp <= 64) RC(grouped_tiles<4>(e, a, ps.n_tiles, s));
+                else if (d.dimp <= 128) RC(grouped_tiles<8>(e, a, ps.n_tiles, s));
+                else RC(grouped_tiles<16>(e, a, ps.n_tiles, s));
             } else {
-                RC(absorbed_attention<T>(e, li, M, s));
+                RC(grouped_rows_bf16<false>(e, li, r, ps.M, s));
             }
-            RC(gemm<T>(e, mp.w_out, w.w_out, ay, L.ld_ay, d.k_out, M, d.n_out, er, s));
+        }
+    } else {
+        RC(run(e, k_qk_rows<T>, dim3(ps.M), LM_THREADS, 0, s, r));
+        const GroupedAttnF32Args a{static_cast<const float*>(r.q), r.c, r.row_slot, r.row_pos, wsp<float>(e, L.ay), L.ld_ay, l.heads, hpg,
+                                   window, l.scale, l.softcap};
+        RC(run(e, k_grouped_attn_f32, dim3(ps.M, l.heads), LM_THREADS, 0, s, a));
+    }
+    return product_out<T>(e, li, ps, s);
+}
+
+template <class T>
+int32_t delta_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
+    const VuibLmConfig& c = e->cfg;
+    const LmLayout& L = e->lay;
+    const VuibLmLayer& l = e->layer[li];
+    const VuibLmDims& d = e->dims[li];
+    const VuibLmLayerWeights& w = e->w[li];
+    RC(mix_in<T>(e, li, ps, s));
+    const DeltaShape ds{l.heads, l.kv_heads, l.dim, d.dimp, l.vdim, d.vdp, l.taps, d.n_ab, d.n_ab, l.scale, l.unit_eps, c.norm_eps};
+    const DeltaWeights dw{w.conv, w.neg_a, w.dt_bias, w.head_norm};
+    const DeltaState st{static_cast<float*>(e->cache[li]), (size_t)d.slot_bytes / 4, (size_t)d.off_v};
+    const int32_t *row_slot = wsp<int32_t>(e, L.row_slot), *row_pos = wsp<int32_t>(e, L.row_pos);
+    const int2* row_ext = wsp<int2>(e, L.row_ext);
+    const DeltaGateArgs<T> ga{ds, dw, st, wsp<float>(e, L.raw), L.ld_raw, wsp<float>(e, L.dout), wsp<T>(e, L.gate), L.ld_gate, wsp<T>(e, L.ay),
+                              L.ld_ay, row_slot, row_pos, row_ext};
+    if (ps.step) {
+        const dim3 grid(l.heads, ps.M);
+        if (d.dimp <= 64) RC(run(e, k_delta_step<T, 16, 1>, grid, DT_THREADS, 0, s, ga));
+        else if (d.dimp <= 128) RC(run(e, k_delta_step<T, 32, 1>, grid, DT_THREADS, 0, s, ga));
+        else RC(run(e, k_delta_step<T, 32, 2>, grid, DT_THREADS, 0, s, ga));
+    } else {
+        const DeltaRowsArgs ra{ds, dw, st, ga.raw, ga.ldraw, wsp<float>(e, L.dx), wsp<float2>(e, L.dg), row_slot, row_pos, row_ext};
+        RC(run(e, k_delta_rows, dim3(ps.M), LM_THREADS, 0, s, ra));
+        const DeltaScanArgs sa{ds, st, ra.out, ra.gates, wsp<int4>(e, L.segs), wsp<float>(e, L.dout)};
+        const int lpc = d.dimp <= 64 ? 16 : 32, cols = DS_THREADS / lpc * DS_CP;
+        const dim3 grid(ps.n_segs, l.heads, (d.vdp + cols - 1) / cols);
+        if (d.dimp <= 64) RC(run(e, k_delta_scan<16, 1>, grid, DS_THREADS, 0, s, sa));
+        else if (d.dimp <= 128) RC(run(e, k_delta_scan<32, 1>, grid, DS_THREADS, 0, s, sa));
+        else RC(run(e, k_delta_scan<32, 2>, grid, DS_THREADS, 0, s, sa));
+        RC(run(e, k_delta_gate<T>, dim3(ps.M), LM_THREADS, 0, s, ga));
+    }
+    return product_out<T>(e, li, ps, s);
+}
+
+// One pass over the layers for the rows whose x, slots and positions are in the workspace.
+template <class T>
+int32_t run_layers(VuibLm* e, Pass ps, cudaStream_t s) {
+    const VuibLmConfig& c = e->cfg;
+    const LmLayout& L = e->lay;
+    ps.few = ps.M <= e->few_rows;
+    for (int li = 0; li < c.n_layers; ++li) {
+        switch (e->layer[li].mixer) {
+            case VUIB_LM_MIX_LATENT: RC(latent_layer<T>(e, li, ps, s)); break;
+            case VUIB_LM_MIX_GROUPED: RC(grouped_layer<T>(e, li, ps, s)); break;
+            default: RC(delta_layer<T>(e, li, ps, s)); break;
         }
         if (e->taps)
-            CK(cudaMemcpy2DAsync(e->taps + (size_t)li * e->R * c.width, (size_t)c.width * 4, x, (size_t)L.ldx * 4,
-                                 (size_t)c.width * 4, M, cudaMemcpyDeviceToDevice, s));
+            CK(cudaMemcpy2DAsync(e->taps + (size_t)li * e->R * c.width, (size_t)c.width * 4, wsp<float>(e, L.x), (size_t)L.ldx * 4,
+                                 (size_t)c.width * 4, ps.M, cudaMemcpyDeviceToDevice, s));
     }
     return VUIB_OK;
 }
@@ -578,10 +803,11 @@ int32_t run_head(VuibLm* e, int M, const int32_t* rows, const int32_t* row_slot,
     const VuibLmConfig& c = e->cfg;
     const LmLayout& L = e->lay;
     T* xn = wsp<T>(e, L.xn);
-    RC(run(e, k_layernorm_rows<T>, dim3(M), 128, 0, s, wsp<float>(e, L.x), L.ldx, c.width, c.norm_eps,
-           LayerNormW{e->head.final_w, e->head.final_b}, xn, LayerNormW{nullptr, nullptr}, static_cast<T*>(nullptr), L.ldx, rows,
-           row_slot, seq_inc, seq_lens));
-    const EpLogitsF32 el{logits, c.vocab};
+    const bool ln = c.block == VUIB_LM_BLOCK_LN2;
+    auto norm = ln ? k_norm_rows<T, true> : k_norm_rows<T, false>;
+    RC(run(e, norm, dim3(M), 128, 0, s, wsp<float>(e, L.x), L.ldx, c.width, c.norm_eps, NormVec{e->head.final_w, ln ? e->head.final_b : nullptr},
+           xn, NormVec{nullptr, nullptr}, static_cast<T*>(nullptr), L.ldx, rows, row_slot, seq_inc, seq_lens));
+    const EpLogitsF32 el{logits, c.vocab, c.logit_scale};
     if (M <= e->few_rows) return few<T>(e, StageRowsT<T>{xn, L.ldx}, el, e->head.head, L.ldx, M, c.vocab, s);
     return gemm<T>(e, e->map_head, e->head.head, xn, L.ldx, L.ldx, M, up(c.vocab, 128), el, s);
 }
@@ -607,6 +833,7 @@ EmbedArgs embed_args(VuibLm* e, const int64_t* tokens) {
     a.vocab = c.vocab;
     a.row_slot = wsp<int32_t>(e, L.row_slot);
     a.row_pos = wsp<int32_t>(e, L.row_pos);
+    a.row_ext = wsp<int2>(e, L.row_ext);
     a.n_slots = c.n_slots;
     a.max_seq = c.max_seq;
     a.flag = wsp<int32_t>(e, L.flag);
@@ -614,14 +841,13 @@ EmbedArgs embed_args(VuibLm* e, const int64_t* tokens) {
 }
 
 template <class T>
-int32_t prefill(VuibLm* e, int n_rows, int n_segs, const std::vector<ExpandGroup>* expand, const int64_t* tokens, int n_want,
-                const int32_t* want, float* logits, cudaStream_t s) {
+int32_t prefill(VuibLm* e, const Pass& ps, const int64_t* tokens, int n_want, const int32_t* want, float* logits, cudaStream_t s) {
     EmbedArgs a = embed_args(e, tokens);
     a.segs = wsp<int4>(e, e->lay.segs);
-    a.n_segs = n_segs;
+    a.n_segs = ps.n_segs;
     a.seq_lens_out = e->seq_lens;
-    RC(run(e, k_lm_embed<T>, dim3(n_rows), 128, 0, s, a));
-    RC(run_layers<T>(e, n_rows, expand, s));
+    RC(run(e, k_lm_embed<T>, dim3(ps.M), 128, 0, s, a));
+    RC(run_layers<T>(e, ps, s));
     for (int w0 = 0; w0 < n_want; w0 += e->R) {
         const int n = n_want - w0 < e->R ? n_want - w0 : e->R;
         RC(run_head<T>(e, n, want + w0, nullptr, nullptr, nullptr, logits + (size_t)w0 * e->cfg.vocab, s));
@@ -635,7 +861,7 @@ int32_t decode(VuibLm* e, int B, const int32_t* slots, const int32_t* seq_inc, c
     a.slots = slots;
     a.seq_lens = e->seq_lens;
     RC(run(e, k_lm_embed<T>, dim3(B), 128, 0, s, a));
-    RC(run_layers<T>(e, B, nullptr, s));
+    RC(run_layers<T>(e, Pass{B, true, 0, 0, nullptr, false}, s));
     return run_head<T>(e, B, nullptr, wsp<int32_t>(e, e->lay.row_slot), seq_inc, e->seq_lens, logits, s);
 }
 
@@ -650,26 +876,40 @@ extern "C" int32_t vuib_lm_create(const VuibLmConfig* cfg, const VuibLmLayer* la
     if (!cfg || !layers || !out) return VUIB_ERR_NULL;
     *out = nullptr;
     const VuibLmConfig& c = *cfg;
-    if (c.dtype != VUIB_LM_BF16 && c.dtype != VUIB_LM_F32) return VUIB_ERR_SHAPE;
+    if ((c.dtype != VUIB_LM_BF16 && c.dtype != VUIB_LM_F32) || (c.block != VUIB_LM_BLOCK_LN2 && c.block != VUIB_LM_BLOCK_RMS)) return VUIB_ERR_SHAPE;
     if (c.vocab < 1 || c.width < 1 || c.n_layers < 1 || c.n_layers > VUIB_LM_MAX_LAYERS || !(c.norm_eps >= 0.f)) return VUIB_ERR_SHAPE;
     if (c.n_slots < 1 || c.max_seq < 1 || c.max_rows < 1 || c.max_rows > 65535 || c.max_prefill_rows < 1) return VUIB_ERR_RANGE;
     for (int i = 0; i < c.n_layers; ++i) {
         const VuibLmLayer& l = layers[i];
-        if (l.mixer != VUIB_LM_MIX_LATENT || (l.mlp != VUIB_LM_MLP_NONE && l.mlp != VUIB_LM_MLP_CLAMPED_GLU)) return VUIB_ERR_SHAPE;
-        if (l.heads < 1 || l.dim < 0 || l.rot_dim < 0 || l.dim + l.rot_dim < 1 || l.vdim < 1 || l.kv_rank < 1 || l.q_rank < 1 ||
-            l.rot_dims < 0 || l.rot_dims > l.rot_dim || l.rot_dims % 2)
-            return VUIB_ERR_SHAPE;
         if (l.mlp != VUIB_LM_MLP_NONE && l.ff < 1) return VUIB_ERR_SHAPE;
-        const VuibLmDims d = layer_dims(c, l);
-        if (c.dtype == VUIB_LM_BF16 ? d.rp > 1024 || latent_attn_smem(d.dp, d.rp, 32, 1) > LM_MAX_SMEM
-                                    : latent_attn_f32_smem(d.dp) > LM_MAX_SMEM)
-            return VUIB_ERR_SHAPE;
+        if (l.heads < 1 || l.dim < 0 || l.vdim < 1) return VUIB_ERR_SHAPE;
+        if (c.block == VUIB_LM_BLOCK_LN2) {
+            if (l.mixer != VUIB_LM_MIX_LATENT || (l.mlp != VUIB_LM_MLP_NONE && l.mlp != VUIB_LM_MLP_CLAMPED_GLU)) return VUIB_ERR_SHAPE;
+            if (l.rot_dim < 0 || l.dim + l.rot_dim < 1 || l.kv_rank < 1 || l.q_rank < 1 || l.rot_dims < 0 || l.rot_dims > l.rot_dim ||
+                l.rot_dims % 2)
+                return VUIB_ERR_SHAPE;
+            const VuibLmDims d = layer_dims(c, l);
+            if (c.dtype == VUIB_LM_BF16 ? d.rp > 1024 || latent_attn_smem(d.dp, d.rp, 32, 1) > LM_MAX_SMEM
+                                        : latent_attn_f32_smem(d.dp) > LM_MAX_SMEM)
+                return VUIB_ERR_SHAPE;
+        } else {
+            if ((l.mixer != VUIB_LM_MIX_GROUPED && l.mixer != VUIB_LM_MIX_DELTA) || (l.mlp != VUIB_LM_MLP_NONE && l.mlp != VUIB_LM_MLP_RELU2))
+                return VUIB_ERR_SHAPE;
+            if (l.dim < 1 || l.kv_heads < 1 || l.heads % l.kv_heads) return VUIB_ERR_SHAPE;
+            if (l.mixer == VUIB_LM_MIX_GROUPED && (l.rot_dims < 0 || l.rot_dims > l.dim || l.rot_dims % 2 || l.window < 0 ||
+                                                   !(l.softcap >= 0.f) || l.dim > GA_MAX_DIM || l.vdim > GA_MAX_DIM))
+                return VUIB_ERR_SHAPE;
+            if (l.mixer == VUIB_LM_MIX_DELTA && (l.taps < 1 || l.dim > DR_MAX_DIM || l.vdim > DR_MAX_VDIM || l.heads > 65535)) return VUIB_ERR_SHAPE;
+        }
     }
     VuibLm* e = new (std::nothrow) VuibLm();
     if (!e) return VUIB_ERR_NULL;
     e->cfg = c;
     e->layer.assign(layers, layers + c.n_layers);
-    for (const VuibLmLayer& l : e->layer) e->dims.push_back(layer_dims(c, l));
+    for (const VuibLmLayer& l : e->layer) {
+        e->dims.push_back(layer_dims(c, l));
+        e->recurrent = e->recurrent || l.mixer == VUIB_LM_MIX_DELTA;
+    }
     e->w.resize(c.n_layers);
     e->maps.resize(c.n_layers);
     e->cache.resize(c.n_layers);
@@ -719,19 +959,22 @@ extern "C" int32_t vuib_lm_bind_workspace(VuibLm* e, void* dev, size_t bytes) {
 extern "C" int32_t vuib_lm_bind_weights(VuibLm* e, const VuibLmHeadWeights* head, const VuibLmLayerWeights* layers) {
     if (!e || !head || !layers) return VUIB_ERR_NULL;
     const VuibLmConfig& c = e->cfg;
-    if (!head->embed || !head->final_w || !head->final_b || !head->head) return fail(e, VUIB_ERR_NULL, "a head weight is NULL");
+    if (!head->embed || !head->final_w || (c.block == VUIB_LM_BLOCK_LN2 && !head->final_b) || !head->head) return fail(e, VUIB_ERR_NULL, "a head weight is NULL");
     for (int i = 0; i < c.n_layers; ++i) {
         const VuibLmLayerWeights& w = layers[i];
         const VuibLmDims& d = e->dims[i];
-        const bool mlp = e->layer[i].mlp != VUIB_LM_MLP_NONE;
-        if (!w.norm1_w || !w.norm1_b || (mlp && (!w.norm2_w || !w.norm2_b)) || !w.q_norm || !w.kv_norm || !w.w_in || !w.w_q || !w.w_uv ||
-            !w.w_out || (d.x_ok && (!w.w_xq || !w.w_xkv)) || (e->layer[i].rot_dims && !w.trig))
-            return fail(e, VUIB_ERR_NULL, "a weight of layer %d is NULL", i);
+        const int mixer = e->layer[i].mixer;
+        bool have = w.norm1_w && w.w_in && w.w_out && (!e->layer[i].rot_dims || w.trig);
+        if (mixer == VUIB_LM_MIX_LATENT)
+            have = have && w.norm1_b && (e->layer[i].mlp == VUIB_LM_MLP_NONE || (w.norm2_w && w.norm2_b)) && w.q_norm && w.kv_norm && w.w_q &&
+                   w.w_uv && (!d.x_ok || (w.w_xq && w.w_xkv));
+        if (mixer == VUIB_LM_MIX_DELTA) have = have && w.conv && w.neg_a && w.dt_bias && w.head_norm;
+        if (!have) return fail(e, VUIB_ERR_NULL, "a weight of layer %d is NULL", i);
         e->w[i] = w;
         if (c.dtype == VUIB_LM_BF16) {
             LmMaps& m = e->maps[i];
-            bool ok = make_map(&m.w_in, w.w_in, d.n_in, d.k_in, 64) && make_map(&m.w_q, w.w_q, d.n_q, d.k_q, 64) &&
-                      make_map(&m.w_out, w.w_out, d.n_out, d.k_out, 64);
+            bool ok = make_map(&m.w_in, w.w_in, d.n_in, d.k_in, 64) && make_map(&m.w_out, w.w_out, d.n_out, d.k_out, 64);
+            if (mixer == VUIB_LM_MIX_LATENT) ok = ok && make_map(&m.w_q, w.w_q, d.n_q, d.k_q, 64);
             if (d.x_ok) ok = ok && make_map(&m.w_xq, w.w_xq, d.n_xq, d.k_q, 64) && make_map(&m.w_xkv, w.w_xkv, d.n_xkv, d.k_kv, 64);
             if (!ok) return fail(e, VUIB_ERR_CUDA, "cuTensorMapEncodeTiled failed for layer %d", i);
         }
@@ -763,6 +1006,12 @@ extern "C" int32_t vuib_lm_prefill(VuibLm* e, int32_t n_segs, const int32_t* slo
     if (n_segs < 1 || n_want < 0) return fail(e, VUIB_ERR_RANGE, "n_segs %d / n_want %d out of range", n_segs, n_want);
     std::vector<int4> segs;
     int rows = 0;
+    if (e->recurrent) {
+        std::vector<int32_t> slots(slot, slot + n_segs);
+        std::sort(slots.begin(), slots.end());
+        if (std::adjacent_find(slots.begin(), slots.end()) != slots.end())
+            return fail(e, VUIB_ERR_RANGE, "a slot appears twice in a call of a model with recurrent layers");
+    }
     for (int i = 0; i < n_segs; ++i) {
         if (slot[i] < 0 || slot[i] >= c.n_slots || pos[i] < 0 || len[i] < 1 || len[i] > c.max_seq || pos[i] > c.max_seq - len[i])
             return fail(e, VUIB_ERR_RANGE, "portion %d: slot %d, positions %d + %d out of range", i, slot[i], pos[i], len[i]);
@@ -773,11 +1022,18 @@ extern "C" int32_t vuib_lm_prefill(VuibLm* e, int32_t n_segs, const int32_t* slo
     }
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     CK(cudaMemcpyAsync(e->ws + e->lay.segs, segs.data(), segs.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
+    const bool forms = c.dtype == VUIB_LM_BF16 && rows >= e->expand_min && rows > e->few_rows;
     std::vector<ExpandGroup> groups;
-    if (e->lay.x_rows && rows >= e->expand_min && rows > e->few_rows) {
+    std::vector<int4> xsegs, tiles;
+    if (forms && c.block == VUIB_LM_BLOCK_RMS) {
+        for (const int4& g : segs)
+            for (int r = (g.z - 1) / GP_TILE * GP_TILE; r >= 0; r -= GP_TILE) {
+                tiles.push_back(make_int4(g.w + r, g.z - r < GP_TILE ? g.z - r : GP_TILE, g.x, g.y + r));
+                tiles.push_back(make_int4(0, 0, 0, 0));
+            }
+    } else if (forms && e->lay.x_rows) {
         // sequences are expanded together while their keys fit the scratch (one sequence always does); tiles with the
         // most keys first
-        std::vector<int4> xsegs, tiles;
         for (const int4& g : segs) {
             const int keys = g.y + g.z;
             if (groups.empty() || groups.back().rows + keys > e->lay.x_rows)
@@ -792,12 +1048,12 @@ extern "C" int32_t vuib_lm_prefill(VuibLm* e, int32_t n_segs, const int32_t* slo
             ++q.n_segs;
             q.rows += keys;
         }
-        CK(cudaMemcpyAsync(e->ws + e->lay.xsegs, xsegs.data(), xsegs.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
-        CK(cudaMemcpyAsync(e->ws + e->lay.tiles, tiles.data(), tiles.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
     }
-    if (c.dtype == VUIB_LM_BF16)
-        return prefill<bf16>(e, rows, n_segs, groups.empty() ? nullptr : &groups, tokens_dev, n_want, want_rows_dev, logits_out_dev, s);
-    return prefill<float>(e, rows, n_segs, nullptr, tokens_dev, n_want, want_rows_dev, logits_out_dev, s);
+    if (!xsegs.empty()) CK(cudaMemcpyAsync(e->ws + e->lay.xsegs, xsegs.data(), xsegs.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
+    if (!tiles.empty()) CK(cudaMemcpyAsync(e->ws + e->lay.tiles, tiles.data(), tiles.size() * sizeof(int4), cudaMemcpyHostToDevice, s));
+    const Pass ps{rows, false, n_segs, (int)tiles.size() / 2, groups.empty() ? nullptr : &groups, false};
+    if (c.dtype == VUIB_LM_BF16) return prefill<bf16>(e, ps, tokens_dev, n_want, want_rows_dev, logits_out_dev, s);
+    return prefill<float>(e, ps, tokens_dev, n_want, want_rows_dev, logits_out_dev, s);
 }
 
 extern "C" int32_t vuib_lm_decode(VuibLm* e, int32_t B, const int32_t* slots_dev, const int32_t* seq_inc_dev,

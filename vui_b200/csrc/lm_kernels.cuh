@@ -84,6 +84,7 @@ __device__ __forceinline__ float2 rotate_pair(float u, float v, float2 cs) {
 }
 
 __device__ __forceinline__ float sigmoid32(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu32(float z) { return z / (1.0f + expf(-z)); }
 
 // ---------------------------------------------------------------------------
 // Embedding rows and the per-row (slot, position) table of the call.
@@ -102,6 +103,7 @@ struct EmbedArgs {
     int n_segs;
     int32_t* row_slot;
     int32_t* row_pos;
+    int2* row_ext;             // rows of the same portion before and after this one
     int32_t* seq_lens_out;     // prefill: the slots' new lengths
     int n_slots, max_seq;
     int32_t* flag;
@@ -114,6 +116,7 @@ static __global__ void __launch_bounds__(128) k_lm_embed(EmbedArgs a) {
     const int r = blockIdx.x;
     if (threadIdx.x == 0) {
         int slot, pos;
+        int2 ext = make_int2(0, 0);
         if (a.slots) {
             slot = a.slots[r];
             if (slot < 0 || slot >= a.n_slots) {
@@ -131,10 +134,12 @@ static __global__ void __launch_bounds__(128) k_lm_embed(EmbedArgs a) {
             const int4 g = a.segs[s];
             slot = g.x;
             pos = g.y + (r - g.w);
+            ext = make_int2(r - g.w, g.w + g.z - 1 - r);
             if (r == g.w + g.z - 1) a.seq_lens_out[slot] = pos + 1;
         }
         a.row_slot[r] = slot;
         a.row_pos[r] = pos;
+        a.row_ext[r] = ext;
     }
     long long tok = a.tokens[r];
     if (tok < 0 || tok >= a.vocab) {
@@ -146,20 +151,20 @@ static __global__ void __launch_bounds__(128) k_lm_embed(EmbedArgs a) {
 }
 
 // ---------------------------------------------------------------------------
-// Layer norm of the fp32 residual with one or two (weight, bias) pairs: a block that reads the same row through two
-// norms needs the mean and the variance once.  Variance is the mean of the squared deviations (two passes).
+// Norm of the fp32 residual with one or two (weight, bias) pairs: a block that reads the same row through two norms
+// needs its statistics once.  CENTER: layer norm, variance as the mean of the squared deviations (two passes);
+// otherwise RMS norm.  A bias may be NULL.
 // ---------------------------------------------------------------------------
-struct LayerNormW {
+struct NormVec {
     const float* w;
     const float* b;
 };
 
-template <class T>
-static __global__ void __launch_bounds__(128) k_layernorm_rows(const float* __restrict__ x, int ldx, int width, float eps,
-                                                               LayerNormW n1, T* __restrict__ out1, LayerNormW n2,
-                                                               T* __restrict__ out2, int ldo, const int32_t* __restrict__ rows,
-                                                               const int32_t* __restrict__ row_slot,
-                                                               const int32_t* __restrict__ seq_inc, int32_t* __restrict__ seq_lens) {
+template <class T, bool CENTER>
+static __global__ void __launch_bounds__(128) k_norm_rows(const float* __restrict__ x, int ldx, int width, float eps, NormVec n1,
+                                                          T* __restrict__ out1, NormVec n2, T* __restrict__ out2, int ldo,
+                                                          const int32_t* __restrict__ rows, const int32_t* __restrict__ row_slot,
+                                                          const int32_t* __restrict__ seq_inc, int32_t* __restrict__ seq_lens) {
     __shared__ float red[32];
     pdl_trigger();
     pdl_wait();
@@ -167,17 +172,19 @@ static __global__ void __launch_bounds__(128) k_layernorm_rows(const float* __re
     const float* xr = x + (size_t)(rows ? rows[r] : r) * ldx;
     constexpr int KEEP = 16;      // the row stays in registers up to 128 * 16 elements
     float v[KEEP];
-    float s[1] = {0.f};
+    float s[1] = {0.f}, mean = 0.f;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
         const int k = threadIdx.x + i * 128;
         v[i] = k < width ? __ldcg(xr + k) : 0.f;
-        s[0] += v[i];
+        if (CENTER) s[0] += v[i];
     }
-    for (int k = threadIdx.x + KEEP * 128; k < width; k += 128) s[0] += __ldcg(xr + k);
-    block_sums<1>(s, red);
-    const float mean = s[0] / (float)width;
-    s[0] = 0.f;
+    if (CENTER) {
+        for (int k = threadIdx.x + KEEP * 128; k < width; k += 128) s[0] += __ldcg(xr + k);
+        block_sums<1>(s, red);
+        mean = s[0] / (float)width;
+        s[0] = 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
         const float d = threadIdx.x + i * 128 < width ? v[i] - mean : 0.f;
@@ -190,8 +197,8 @@ static __global__ void __launch_bounds__(128) k_layernorm_rows(const float* __re
     block_sums<1>(s, red);
     const float rstd = 1.0f / sqrtf(s[0] / (float)width + eps);
     auto put = [&](int k, float d) {
-        Store<T>::put(out1 + (size_t)r * ldo + k, fmaf(d * rstd, __ldg(n1.w + k), __ldg(n1.b + k)));
-        if (out2) Store<T>::put(out2 + (size_t)r * ldo + k, fmaf(d * rstd, __ldg(n2.w + k), __ldg(n2.b + k)));
+        Store<T>::put(out1 + (size_t)r * ldo + k, fmaf(d * rstd, __ldg(n1.w + k), n1.b ? __ldg(n1.b + k) : 0.f));
+        if (out2) Store<T>::put(out2 + (size_t)r * ldo + k, fmaf(d * rstd, __ldg(n2.w + k), n2.b ? __ldg(n2.b + k) : 0.f));
     };
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
@@ -392,24 +399,64 @@ struct EpPre<EpRotatedQ<T>> {
     }
 };
 
+// Everything a block with one norm reads from x: the mixer's fp32 rows [0, n_raw) (a bias may be added), its gate rows
+// [n_raw, n_gate) through silu, then the MLP's units through the square of relu.
+template <class T>
+struct EpMixIn {
+    int n_raw, n_gate, n_mlp, ff;
+    const float* bias;        // (n_raw) or NULL
+    float* raw; int ldraw;
+    T* gate; int ldgate;
+    T* act; int ldact;        // columns up to a multiple of 64
+    __device__ __forceinline__ void put(int m, int n, float v0, float v1, float2 b) const {
+        if (n < n_raw) {
+            *reinterpret_cast<float2*>(raw + (size_t)m * ldraw + n) = make_float2(v0 + b.x, v1 + b.y);
+        } else if (n < n_gate) {
+            Store<T>::put2(gate + (size_t)m * ldgate + (n - n_raw), silu32(v0), silu32(v1));
+        } else if (n >= n_mlp && n - n_mlp < ff) {
+            const float r0 = fmaxf(v0, 0.f), r1 = fmaxf(v1, 0.f);
+            Store<T>::put2(act + (size_t)m * ldact + (n - n_mlp), r0 * r0, r1 * r1);
+        }
+    }
+    __device__ __forceinline__ float2 bias_at(int n) const {
+        return bias && n < n_raw ? __ldg(reinterpret_cast<const float2*>(bias + n)) : make_float2(0.f, 0.f);
+    }
+    __device__ __forceinline__ void store(int m, int n, float v0, float v1) const { put(m, n, v0, v1, bias_at(n)); }
+};
+
+template <class T>
+struct EpPre<EpMixIn<T>> {
+    typedef float2 type;
+    static __device__ __forceinline__ int ask(const EpMixIn<T>&, int) { return 0; }
+    static __device__ __forceinline__ float2 pre(const EpMixIn<T>& ep, int, int n) { return ep.bias_at(n); }
+    static __device__ __forceinline__ void store(const EpMixIn<T>& ep, int m, int n, float v0, float v1, const float2& b) { ep.put(m, n, v0, v1, b); }
+};
+
 // x += W a in 32 bits.  Every element is added to once per launch, so the reductions have no order to depend on; they
 // return nothing, so no thread waits for the old value.
 struct EpAddResidual {
     float* x; int ldx, N;
+    const float* bias;        // (N up to even) or NULL
     __device__ __forceinline__ void store(int m, int n, float v0, float v1) const {
         float* p = x + (size_t)m * ldx + n;
+        if (bias && n < N) {
+            const float2 b = __ldg(reinterpret_cast<const float2*>(bias + n));
+            v0 += b.x;
+            v1 += b.y;
+        }
         if (n + 1 < N) asm volatile("red.global.add.v2.f32 [%0], {%1, %2};" ::"l"(p), "f"(v0), "f"(v1) : "memory");
         else if (n < N) atomicAdd(p, v0);
     }
 };
 
-// fp32 rows (logits).
+// fp32 rows times a constant (logits).
 struct EpLogitsF32 {
     float* out; int N;
+    float scale;
     __device__ __forceinline__ void store(int m, int n, float v0, float v1) const {
         float* p = out + (size_t)m * N + n;
-        if (n < N) p[0] = v0;
-        if (n + 1 < N) p[1] = v1;
+        if (n < N) p[0] = v0 * scale;
+        if (n + 1 < N) p[1] = v1 * scale;
     }
 };
 
@@ -485,7 +532,7 @@ template <class T>
 struct StageLayerNorm2 {
     const float* x; int ldx, width;
     float eps;
-    LayerNormW n1, n2;
+    NormVec n1, n2;
     int split;
     const int32_t* rows;      // optional gather of x's rows
     static __host__ __device__ size_t smem(int RT, int K) { return (size_t)RT * K * (2 * sizeof(T) + 4); }
@@ -617,14 +664,13 @@ struct StageLayerNorm2 {
     __device__ __forceinline__ int tile_of(int n) const { return n >= split ? 1 : 0; }
 };
 
-// RMSNorm of an fp32 row (the queries' latent); the grid's last CTA appends the call's cache rows.
+// RMS norm of an fp32 row; its padding up to a multiple of 4 may be read.
 template <class T>
-struct StageLatentQ {
-    const float* dq; int lddq, q_rank;
+struct StageRms {
+    const float* x; int ldx, width;
     float eps;
     const float* norm_w;
-    LatentRow lat;
-    static constexpr bool HAS_EXTRA = true;
+    static constexpr bool HAS_EXTRA = false;
     static __host__ __device__ size_t smem(int RT, int K) { return (size_t)RT * K * sizeof(T); }
     template <int RT>
     __device__ __forceinline__ void stage(unsigned char* sm, float* red, int K, int r0, int nr) const {
@@ -634,8 +680,8 @@ struct StageLatentQ {
         for (int r = 0; r < RT; ++r) {
             s[r] = 0.f;
             if (r < nr)
-                for (int k = threadIdx.x; k < q_rank; k += LM_THREADS) {
-                    const float v = __ldcg(dq + (size_t)(r0 + r) * lddq + k);
+                for (int k = threadIdx.x; k < width; k += LM_THREADS) {
+                    const float v = __ldcg(x + (size_t)(r0 + r) * ldx + k);
                     s[r] = fmaf(v, v, s[r]);
                 }
         }
@@ -644,40 +690,45 @@ struct StageLatentQ {
 #pragma unroll
             for (int r = 0; r < RT; ++r) {
                 float o = 0.f;
-                if (k < q_rank && r < nr)
-                    o = __ldcg(dq + (size_t)(r0 + r) * lddq + k) * (1.0f / sqrtf(s[r] / (float)q_rank + eps)) * __ldg(norm_w + k);
+                if (k < width && r < nr)
+                    o = __ldcg(x + (size_t)(r0 + r) * ldx + k) * (1.0f / sqrtf(s[r] / (float)width + eps)) * __ldg(norm_w + k);
                 Store<T>::put(X + r * K + k, o);
             }
     }
     template <int RT>
     __device__ __forceinline__ const T* tile(const unsigned char* sm, int, int) const { return reinterpret_cast<const T*>(sm); }
-    __device__ __forceinline__ void extra(int M) const {
-        for (int m = threadIdx.x >> 5; m < M; m += LM_WARPS) latent_row<T>(lat, m, threadIdx.x & 31);
-    }
+    __device__ __forceinline__ void extra(int) const {}
     static constexpr int TILES = 1;
     static constexpr bool K_PARTS = false;
     static __host__ __device__ size_t scratch(int RT, int K) { return (size_t)(RT + 1) * K * 4; }
     __device__ __forceinline__ void constants(float* sc, int K) const {
-        for (int k = threadIdx.x; k < K; k += LM_THREADS) sc[k] = k < q_rank ? __ldg(norm_w + k) : 0.f;
+        for (int k = threadIdx.x; k < K; k += LM_THREADS) sc[k] = k < width ? __ldg(norm_w + k) : 0.f;
     }
     template <int RT>
     __device__ __forceinline__ void stage_rows(bf16* X, int ld, float* red, float* sc, int K, int M, int) const {
         constexpr int WPR = LM_WARPS / RT, TPR = 32 * WPR, U = 4;
         const int r = threadIdx.x / TPR, i0 = threadIdx.x % TPR, warp = threadIdx.x >> 5;
         const bool on = r < M;
-        const float* src = dq + (size_t)(on ? r : 0) * lddq;
+        const float* src = x + (size_t)(on ? r : 0) * ldx;
         float* xs = sc + (size_t)(1 + r) * K;
+        const int nv = (width + 3) / 4;
         float ss = 0.f;
-        for (int k0 = i0; k0 < K; k0 += U * TPR) {
-            float v[U];
-#pragma unroll
-            for (int u = 0; u < U; ++u) v[u] = k0 + u * TPR < q_rank ? __ldcg(src + k0 + u * TPR) : 0.f;
+        for (int q0 = i0; q0 < K / 4; q0 += U * TPR) {
+            float4 v[U];
 #pragma unroll
             for (int u = 0; u < U; ++u)
-                if (k0 + u * TPR < K) {
-                    xs[k0 + u * TPR] = v[u];
-                    ss = fmaf(v[u], v[u], ss);
+                v[u] = q0 + u * TPR < nv ? __ldcg(reinterpret_cast<const float4*>(src) + q0 + u * TPR) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int q = q0 + u * TPR;
+                if (q < K / 4) {
+                    if (4 * q + 1 >= width) v[u].y = 0.f;     // what lies beyond the row is not part of it
+                    if (4 * q + 2 >= width) v[u].z = 0.f;
+                    if (4 * q + 3 >= width) v[u].w = 0.f;
+                    reinterpret_cast<float4*>(xs)[q] = v[u];
+                    ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, ss))));
                 }
+            }
         }
         ss = warp_sum(ss);
         if ((threadIdx.x & 31) == 0) red[warp] = ss;
@@ -686,11 +737,24 @@ struct StageLatentQ {
 #pragma unroll
         for (int w = 0; w < WPR; ++w) ss += red[r * WPR + w];
         if (!on) return;
-        const float rinv = 1.0f / sqrtf(ss / (float)q_rank + eps);
-        for (int k = 2 * i0; k < K; k += 2 * TPR)
-            Store<bf16>::put2(X + (size_t)r * ld + k, xs[k] * rinv * sc[k], xs[k + 1] * rinv * sc[k + 1]);
+        const float rinv = 1.0f / sqrtf(ss / (float)width + eps);
+        for (int q = i0; q < K / 4; q += TPR) {
+            const float4 v = reinterpret_cast<const float4*>(xs)[q], w = reinterpret_cast<const float4*>(sc)[q];
+            Store<bf16>::put2(X + (size_t)r * ld + 4 * q, v.x * rinv * w.x, v.y * rinv * w.y);
+            Store<bf16>::put2(X + (size_t)r * ld + 4 * q + 2, v.z * rinv * w.z, v.w * rinv * w.w);
+        }
     }
     __device__ __forceinline__ int tile_of(int) const { return 0; }
+};
+
+// The same of the queries' latent; the grid's last CTA appends the call's cache rows.
+template <class T>
+struct StageLatentQ : StageRms<T> {
+    LatentRow lat;
+    static constexpr bool HAS_EXTRA = true;
+    __device__ __forceinline__ void extra(int M) const {
+        for (int m = threadIdx.x >> 5; m < M; m += LM_WARPS) latent_row<T>(lat, m, threadIdx.x & 31);
+    }
 };
 
 template <class T>

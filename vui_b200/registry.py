@@ -62,3 +62,4 @@ def open_engine(model, **kw):
 
 register(SPEECH, ".model:VuiB200", ".engine:Engine")
 register("Vidotar", ".token_lm:Vidotar", ".token_engine:TokenEngine")
+register("Medirax", ".token_lm:Medirax", ".token_engine:TokenEngine")

@@ -15,7 +15,7 @@ from torch import Tensor
 
 from . import _lib
 from .slots import SlotEngine, _get_bucket, _ptr
-from .token_lm import TokenLM, abi_layer, trig_table
+from .token_lm import GroupedMixer, TokenLM, abi_config, abi_layers, trig_table
 
 DEFAULT_MAX_SEQ = 2048
 
@@ -102,12 +102,11 @@ class TokenEngine(SlotEngine):
         m, dev, c = self.model, self.device, self.model.config
         n_slots = self.max_rows + 1
         b16 = m.dtype == torch.bfloat16
-        cfg = _lib.VuibLmConfig(c.vocab, c.width, len(c.layers), _lib.LM_BF16 if b16 else _lib.LM_F32, n_slots, self.max_seq,
-                                self.max_rows, self.max_prefill_rows, c.norm_eps, c.embed_scale)
-        layers = (_lib.VuibLmLayer * len(c.layers))(*[abi_layer(s) for s in c.layers])
-        _lib.check(None, self._lib.vuib_lm_create(C.byref(cfg), layers, C.byref(self._handle)))
-        dims = []
-        for i in range(len(c.layers)):
+        cfg = abi_config(c, dtype=_lib.LM_BF16 if b16 else _lib.LM_F32, n_slots=n_slots, max_seq=self.max_seq, max_rows=self.max_rows,
+                         max_prefill_rows=self.max_prefill_rows)
+        _lib.check(None, self._lib.vuib_lm_create(C.byref(cfg), abi_layers(c), C.byref(self._handle)))
+        dims = []                       # per run of a layer
+        for i in range(len(c.runs)):
             d = _lib.VuibLmDims()
             self._ck(self._lib.vuib_lm_layer_dims(self._handle, i, C.byref(d)))
             dims.append(d)
@@ -116,23 +115,29 @@ class TokenEngine(SlotEngine):
         self._ws = torch.zeros(nbytes.value + 256, device=dev, dtype=torch.uint8)
         ws_ptr = (self._ws.data_ptr() + 255) & ~255
         self._ck(self._lib.vuib_lm_bind_workspace(self._handle, C.c_void_p(ws_ptr), nbytes.value))
-        # one cached row per position and layer
-        self.cache = [torch.zeros(n_slots, self.max_seq, d.dp, device=dev, dtype=m.dtype) for d in dims]
+        # what a slot holds per run of a layer: cached rows, key/value rings, or recurrent state
+        self.cache = [torch.zeros(n_slots, d.slot_bytes, device=dev, dtype=torch.uint8) for d in dims]
+        # positions a slot's shortest ring holds beyond its window (None: every position is kept)
+        spare = [d.cap - s.window for d, s in zip(dims, (c.layers[i].mixer for i in c.runs))
+                 if isinstance(s, GroupedMixer) and d.cap < self.max_seq]
+        self._ring_spare = min(spare) if spare else None
+        self._ring_top = [0] * n_slots   # the most positions a slot has held since it was taken
         self.seq_lens = torch.zeros(n_slots, device=dev, dtype=torch.int32)
         ptrs = (C.c_void_p * len(self.cache))(*[t.data_ptr() for t in self.cache])
         self._ck(self._lib.vuib_lm_bind_cache(self._handle, ptrs, C.c_void_p(self.seq_lens.data_ptr())))
-        head, packed = m.packed(dims)
+        head, packed = m.packed([dims[c.runs.index(i)] if i in c.runs else None for i in range(len(c.layers))])
         self._trig: dict[tuple[float, int], Tensor] = {}
-        lw = (_lib.VuibLmLayerWeights * len(packed))()
-        for i, (p, s) in enumerate(zip(packed, c.layers)):
-            for k, t in p.items():
+        lw = (_lib.VuibLmLayerWeights * len(c.runs))()
+        for i, n in enumerate(c.runs):
+            for k, t in packed[n].items():
                 setattr(lw[i], k, t.data_ptr())
-            if s.mixer.rot_dims:
-                key = (s.mixer.rot_base, s.mixer.rot_dims)
+            mixer = c.layers[n].mixer
+            if mixer.rot_dims:
+                key = (mixer.rot_base, mixer.rot_dims)
                 if key not in self._trig:
                     self._trig[key] = trig_table(*key, self.max_seq).to(dev)
                 lw[i].trig = self._trig[key].data_ptr()
-        hw = _lib.VuibLmHeadWeights(*[head[k].data_ptr() for k in ("embed", "final_w", "final_b", "head")])
+        hw = _lib.VuibLmHeadWeights(**{k: t.data_ptr() for k, t in head.items()})
         self._ck(self._lib.vuib_lm_bind_weights(self._handle, C.byref(hw), lw))
         # static I/O of the captured steps
         N = self.max_rows
@@ -148,10 +153,26 @@ class TokenEngine(SlotEngine):
     def _set_len(self, slot: int, n: int) -> None:
         super()._set_len(slot, n)
         self._len[slot] = n
+        if n == 0:
+            self._ring_top[slot] = 0
+
+    def _grow(self, slot: int, n: int) -> None:
+        """The host's count of a slot's positions, after a call that appended to it."""
+        self._len[slot] = n
+        self._ring_top[slot] = max(self._ring_top[slot], n)
+
+    def _rewind_row(self, row, offset: int) -> int:
+        if 0 < offset < row.offset:
+            if self.model.config.recurrent:
+                raise ValueError("recurrent state cannot be taken back: rewind to 0")
+            if self._ring_spare is not None and self._ring_top[row.idx] - offset >= self._ring_spare:
+                raise ValueError(f"the keys that position {offset} sees are no longer held")
+        return super()._rewind_row(row, offset)
 
     def reset(self) -> None:
         super().reset()
         self._len = [0] * (self.max_rows + 1)
+        self._ring_top = [0] * (self.max_rows + 1)
 
     # --------------------------------------------------------------- sampling
     def _apply_cfg(self, cfg: TokenGenConfig) -> None:
@@ -219,7 +240,7 @@ class TokenEngine(SlotEngine):
             self._g_tokens[:n] = torch.tensor([ids[0] for _, ids, _, _ in single], device=self.device)
             self._decode_replay(n, False)
             for k, (row, _, want, a) in enumerate(single):
-                self._len[row.idx] += 1
+                self._grow(row.idx, row.offset + 1)
                 if want:
                     out[a:a + len(want)] = self._g_logits[k]
         if portions:
@@ -249,7 +270,7 @@ class TokenEngine(SlotEngine):
             self._ck(self._lib.vuib_lm_prefill(self._handle, n, slot, pos, ln, _ptr(tokens), len(want), _ptr(rows), _ptr(logits),
                                                self._stream))
             for s, p, t, _ in pend:
-                self._len[s] = p + t.shape[0]
+                self._grow(s, p + t.shape[0])
             if want:
                 out[torch.tensor(dst, device=self.device)] = logits
 
@@ -308,7 +329,7 @@ class TokenEngine(SlotEngine):
             self._decode_replay(n, True)
             done = []
             for s, (row, ri), tok in zip(slots, states, self._read_tokens(n)):
-                self._len[s] += 1
+                self._grow(s, row.offset + 1)
                 if not goes_on(row, ri, tok):
                     done.append(s)
             if done:
@@ -336,4 +357,4 @@ class TokenEngine(SlotEngine):
             self._g_tokens[0] = tok
             self._decode_replay(1, True)
             tok = self._read_tokens(1)[0]
-            self._len[row.idx] += 1
+            self._grow(row.idx, row.offset + 1)
