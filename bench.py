@@ -23,9 +23,9 @@ Under torchrun (N > 1) every rank is an independent replica with its own streams
 on its own GPU; there is no data-path collective, the process group only aligns
 the timed window and takes the max time over ranks.
 
-`--token-model` times the token model's prefill and decode at several sizes beside the speech backbone at equal size
+`--token-model` times the token models' prefill and decode at several sizes beside the speech backbone at equal size
 (a JSON line of its own, nothing of the default workload); `--profile-token-model B` runs one decode step of B rows and one
-prefill of both models kernel by kernel and exits.
+prefill of the models kernel by kernel and exits.
 
 `--impl reference` times the CPU restatement of the reference's PyTorch path
 (oracle/, fp32, all host threads) on the same metric.  `--profile-frames N` runs N
@@ -665,7 +665,7 @@ def lm_model(size, dev):
                     kv_rank=size["kv_rank"], scale=(size["dim"] + size["rot_dim"]) ** -0.5, rot_base=10000.0,
                     rot_dims=size["rot_dim"])
     layers = (LayerSpec(m, ClampedGLU(ff=size["ff"], limit=7.0)),) * size["layers"]
-    return Vidotar.random_init(TokenLMConfig(LM_VOCAB, size["width"], 1e-5, 1.0, layers), seed=0, device=dev)
+    return Vidotar.random_init(TokenLMConfig(LM_VOCAB, size["width"], 1e-5, layers), seed=0, device=dev)
 
 
 def backbone_model(size, dev):
@@ -707,20 +707,36 @@ class ColdTimer:
         return statistics.median(times)
 
 
+def medirax_model(size, dev):
+    """Delta and attention layers in turn; attention with the backbone's heads, delta heads of 128 x 128."""
+    from vui_b200.token_lm import DeltaMixer, GroupedMixer, LayerSpec, Medirax, SquaredReLU, TokenLMConfig
+
+    h, n = size["heads"], size["width"] // 128
+    attn = GroupedMixer(heads=h, kv_heads=h // 2, dim=size["dim"], vdim=size["dim"], scale=size["dim"] ** -0.5, rot_base=10000.0,
+                        rot_dims=size["dim"], window=1024, softcap=30.0)
+    delta = DeltaMixer(heads=n, kv_heads=n // 2, dim=128, vdim=128, taps=4, scale=128 ** -0.5)
+    layers = tuple(LayerSpec(delta if i % 2 == 0 else attn, SquaredReLU(ff=size["ff"])) for i in range(size["layers"]))
+    return Medirax.random_init(TokenLMConfig(LM_VOCAB, size["width"], 1e-5, layers, block="rms"), seed=0, device=dev)
+
+
 class LmBench:
-    """The token model's engine at fixed context, and what its decode and prefill move and multiply."""
+    """A token model's engine at fixed context, and what its decode and prefill move and multiply."""
 
     def __init__(self, size, dev, rows, ctx, prefill_rows):
         import torch
 
         from vui_b200 import TokenEngine
 
-        self.size, self.ctx = size, ctx
-        self.model = lm_model(size, dev)
+        self.size, self.ctx, self.torch = size, ctx, torch
+        self.model = self.make(size, dev)
         self.eng = TokenEngine(model=self.model, max_rows=rows, max_seq=2048, max_prefill_rows=prefill_rows)
-        for c in self.eng.cache:
-            c[..., : size["kv_rank"]].normal_()
-        self.torch = torch
+        for c, i in zip(self.eng.cache, self.model.config.runs):
+            self.fill(c, self.model.config.layers[i].mixer)
+
+    make = staticmethod(lm_model)
+
+    def fill(self, cache, mixer):
+        cache.view(self.torch.bfloat16).normal_()
 
     def rewind(self, n):
         self.eng.seq_lens.fill_(n)
@@ -753,6 +769,40 @@ class LmBench:
         per_tok = 2 * (sum(t.numel() for k, t in self.model.sd.items() if t.dim() == 2 and k not in ("embed", "head")))
         attn = z["layers"] * z["heads"] * n_tok * (n_tok + 1) * (z["dim"] + z["rot_dim"] + z["vdim"])
         return n_seq * (n_tok * per_tok + attn)
+
+
+class MediraxBench(LmBench):
+    make = staticmethod(medirax_model)
+
+    def fill(self, cache, mixer):
+        if hasattr(mixer, "taps"):
+            cache.view(self.torch.float32).normal_(0.0, 0.05)
+        else:
+            super().fill(cache, mixer)
+
+    def mixers(self):
+        c = self.model.config
+        return [c.layers[i].mixer for i in c.runs]
+
+    def decode_bytes(self, B):
+        b = 0
+        for m in self.mixers():
+            if hasattr(m, "taps"):
+                b += 2 * 4 * m.heads * m.dim * m.vdim          # the state, read and written
+            else:
+                b += 2 * min(self.ctx + 1, m.window) * m.kv_heads * (m.dim + m.vdim)
+        return self.model.weight_bytes_per_step() + B * b
+
+    def prefill_flops(self, n_seq, n_tok):
+        per_tok = 2 * sum(t.numel() for k, t in self.model.sd.items() if t.dim() == 2 and k not in ("embed", "head"))
+        mix = 0
+        for m in self.mixers():
+            if hasattr(m, "taps"):
+                mix += n_tok * 6 * m.heads * m.dim * m.vdim    # S^T k, k u^T, S^T q
+            else:
+                pairs = sum(min(i + 1, m.window) for i in range(n_tok))
+                mix += 2 * pairs * m.heads * (m.dim + m.vdim)
+        return n_seq * (n_tok * per_tok + mix)
 
 
 class BackboneBench:
@@ -831,7 +881,7 @@ def token_model_bench(args):
         if args.token_sizes and name not in args.token_sizes.split(","):
             continue
         res[name] = {}
-        for label, cls in (("vidotar", LmBench), ("vui_backbone", BackboneBench)):
+        for label, cls in (("vidotar", LmBench), ("medirax", MediraxBench), ("vui_backbone", BackboneBench)):
             if label == "vui_backbone" and size["width"] > 1536:
                 continue
             b = cls(size, dev, 64, ctx, 4096)
@@ -860,12 +910,12 @@ def token_model_bench(args):
 
 
 def profile_token_model(args):
-    """One eager decode step of B rows and one prefill of 16 x 256 of both models at 1024x24 (4 layers of it)."""
+    """One eager decode step of B rows and one prefill of 16 x 256 of the models at 1024x24 (4 layers of it)."""
     import torch
 
     dev = torch.device("cuda", 0)
     size = dict(LM_SIZES["1024x24"], layers=2)
-    for cls in (LmBench, BackboneBench):
+    for cls in (LmBench, MediraxBench, BackboneBench):
         b = cls(size, dev, max(args.profile_token_model, 16), 512, 4096)
         B = args.profile_token_model
         for _ in range(2):
@@ -1030,7 +1080,7 @@ def main():
     ap.add_argument("--profile-frames", type=int, default=0, help="run N frames without a graph and exit (for ncu)")
     ap.add_argument("--profile-codec", type=int, default=0, help="run N streamed codec frames without a graph and exit")
     ap.add_argument("--profile-encoder", type=int, default=0, help="run N codec-encoder calls on a 10 s buffer and exit")
-    ap.add_argument("--token-model", action="store_true", help="token model prefill / decode beside the speech backbone, and exit")
+    ap.add_argument("--token-model", action="store_true", help="the token models' prefill / decode beside the speech backbone, and exit")
     ap.add_argument("--token-sizes", default="", help="with --token-model: sizes to run, separated by commas")
     ap.add_argument("--profile-token-model", type=int, default=0, metavar="B", help="one decode step of B rows and one prefill, and exit")
     args = ap.parse_args()
