@@ -13,10 +13,19 @@
 // position 0 starts from zeros, whatever the slot held before.
 //
 //   decode          k_delta_step: convolution, unit norms, gates, state, output norm and gate of one head and row.
-//   many rows       k_delta_rows (convolution, unit norms, gates), then k_delta_scan (token by token) or the chunked form,
-//                   then k_delta_gate (output norm and gate, the ring's new rows).
+//   many rows       k_delta_rows (convolution, unit norms, gates), the recurrence, then k_delta_gate (output norm and gate, the
+//                   ring's new rows).  The recurrence runs token by token (k_delta_scan) or in chunks.
+//
+// Chunks of 64 tokens (bf16 models).  With G_t the sum of the log decays from the chunk's start to t and S_0 the state before
+// it, unrolling the recurrence gives a unit lower triangular system for the chunk's writes,
+//   (1 + A) u = beta v - (beta e^G k) S_0,   A_ts = beta_t e^(G_t - G_s) k_t . k_s  (s < t),
+//   o_t = e^(G_t) S_0^T q_t + sum_{s <= t} e^(G_t - G_s) (k_s . q_t) u_s,   S_0' = e^(G_C) S_0 + sum_s e^(G_C - G_s) k_s u_s^T.
+// k_delta_solve does what does not need S_0, every chunk on its own: it solves the system for U (right side beta v) and W
+// (right side beta e^G k) by substitution in fp32, and leaves P_ts = e^(G_t - G_s) q_t . k_s.  k_delta_chunks then carries the state
+// from chunk to chunk: u = U - W S_0, o and S_0' as above.  The state stays in fp32 accumulators; a bf16 MMA takes a 32-bit
+// operand as hi + lo bf16 pairs, three products per pair of operands (the product of the two low parts is left out).
 #pragma once
-#include "lm_kernels.cuh"
+#include "latent_attn.cuh"
 
 namespace vuib {
 
@@ -88,6 +97,9 @@ struct DeltaRowsArgs {
     const int2* row_ext;
 };
 
+// One row per CTA, any size.  SPLIT: queries and keys are left as bf16, a head's dimp high parts and then its dimp low parts,
+// in the space of its floats.
+template <bool SPLIT>
 static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows(DeltaRowsArgs a) {
     pdl_trigger();
     pdl_wait();
@@ -109,10 +121,94 @@ static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows(DeltaRowsArgs 
         const float r = 1.0f / sqrtf(warp_sum(ss) + d.unit_eps) * (i < d.G ? d.scale : 1.0f);
 #pragma unroll
         for (int j = 0; j < P; ++j)
-            if (lane + 32 * j < d.dimp) out[i * d.dimp + lane + 32 * j] = v[j] * r;
+            if (lane + 32 * j < d.dimp) {
+                const int c = lane + 32 * j;
+                if (SPLIT) {
+                    bf16* o = reinterpret_cast<bf16*>(out + i * d.dimp);
+                    const bf16 hi = f2bf(v[j] * r);
+                    o[c] = hi;
+                    o[d.dimp + c] = f2bf(v[j] * r - bf2f(hi));
+                } else {
+                    out[i * d.dimp + c] = v[j] * r;
+                }
+            }
     }
     for (int c = 2 * d.G * d.dimp + threadIdx.x; c < d.C; c += LM_THREADS) out[c] = delta_conv(d, a.w, raw, a.ldraw, ring, pos, back, c);
     for (int h = threadIdx.x; h < d.H; h += LM_THREADS) a.gates[(size_t)m * d.H + h] = delta_gates(d, a.w, raw, h);
+}
+
+// DR_ROWS consecutive rows per CTA for up to DR_TAPS taps and heads of up to 128: the rows a convolution shares are read once.
+constexpr int DR_ROWS = 8, DR_TAPS = 4;
+
+template <bool SPLIT>
+static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows_tile(DeltaRowsArgs a, int M) {
+    __shared__ int row_s[DR_ROWS], pos_s[DR_ROWS], back_s[DR_ROWS];
+    pdl_trigger();
+    const DeltaShape& d = a.d;
+    const int m0 = blockIdx.x * DR_ROWS, nr = min(DR_ROWS, M - m0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_wait();
+    if (threadIdx.x < DR_ROWS) {
+        const int m = m0 + min((int)threadIdx.x, nr - 1);
+        row_s[threadIdx.x] = __ldcg(a.row_slot + m);
+        pos_s[threadIdx.x] = __ldcg(a.row_pos + m);
+        back_s[threadIdx.x] = __ldcg(&a.row_ext[m].x);
+    }
+    __syncthreads();
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int vblocks = (d.H * d.vdp + 127) / 128;
+    for (int i = warp; i < 2 * d.G + vblocks; i += LM_WARPS) {
+        const bool unit = i < 2 * d.G;      // a query or key head; else 128 value columns
+        const int c = unit ? i * d.dimp + 4 * lane : 2 * d.G * d.dimp + (i - 2 * d.G) * 128 + 4 * lane;
+        const bool in = unit ? 4 * lane < d.dimp : c < d.C;
+        float4 x[DR_ROWS + DR_TAPS - 1], w[DR_TAPS];
+#pragma unroll
+        for (int r = 0; r < DR_ROWS + DR_TAPS - 1; ++r) {
+            const int m = m0 + r - (DR_TAPS - 1);
+            x[r] = in && m >= 0 && m < M ? __ldcg(reinterpret_cast<const float4*>(a.raw + (size_t)m * a.ldraw + c)) : zero;
+        }
+#pragma unroll
+        for (int j = 0; j < DR_TAPS; ++j)   // w[j] multiplies the row j back
+            w[j] = in && j < d.taps ? __ldg(reinterpret_cast<const float4*>(a.w.conv + (size_t)(d.taps - 1 - j) * d.C + c)) : zero;
+#pragma unroll
+        for (int r = 0; r < DR_ROWS; ++r) {
+            if (r >= nr) break;
+            const int back = back_s[r], pos = pos_s[r];
+            float4 y = zero;
+#pragma unroll
+            for (int j = DR_TAPS - 1; j >= 0; --j) {
+                float4 v = x[r + DR_TAPS - 1 - j];
+                if (j > back)                // before the portion: the ring, or nothing before the start
+                    v = in && j < d.taps && j <= pos
+                            ? __ldcg(reinterpret_cast<const float4*>(a.st.ring(row_s[r]) + (size_t)((pos - j) % d.taps) * d.C + c)) : zero;
+                y.x = fmaf(v.x, w[j].x, y.x);
+                y.y = fmaf(v.y, w[j].y, y.y);
+                y.z = fmaf(v.z, w[j].z, y.z);
+                y.w = fmaf(v.w, w[j].w, y.w);
+            }
+            y = make_float4(silu32(y.x), silu32(y.y), silu32(y.z), silu32(y.w));
+            float* out = a.out + (size_t)(m0 + r) * d.C + (unit ? i * d.dimp : c);
+            if (unit) {
+                const float ss = warp_sum(fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w))));
+                const float n = 1.0f / sqrtf(ss + d.unit_eps) * (i < d.G ? d.scale : 1.0f);
+                y = make_float4(y.x * n, y.y * n, y.z * n, y.w * n);
+                if (SPLIT && in) {
+                    uint2 hi, lo;
+                    split_bf16x2(y.x, y.y, hi.x, lo.x);
+                    split_bf16x2(y.z, y.w, hi.y, lo.y);
+                    reinterpret_cast<uint2*>(out)[lane] = hi;
+                    reinterpret_cast<uint2*>(out + d.dimp / 2)[lane] = lo;
+                } else if (in) {
+                    reinterpret_cast<float4*>(out)[lane] = y;
+                }
+            } else if (in) {
+                *reinterpret_cast<float4*>(out) = y;
+            }
+        }
+    }
+    for (int i = threadIdx.x; i < nr * d.H; i += LM_THREADS) {
+        const int r = i / d.H, h = i - r * d.H;
+        a.gates[(size_t)(m0 + r) * d.H + h] = delta_gates(d, a.w, a.raw + (size_t)(m0 + r) * a.ldraw, h);
+    }
 }
 
 // ---------------------------------------------------------------------------
@@ -215,6 +311,388 @@ static __global__ void __launch_bounds__(DS_THREADS) k_delta_scan(DeltaScanArgs 
 #pragma unroll
             for (int i = 0; i < NV; ++i)
                 if (sub + i * LPC < nv) *(reinterpret_cast<float4*>(S + (size_t)c * d.dimp) + sub + i * LPC) = s[c][i];
+}
+
+// ---------------------------------------------------------------------------
+// The chunked form.
+// ---------------------------------------------------------------------------
+constexpr int DC_ROWS = 64;
+constexpr int DC_MAX_DIM = 128;   // padded key size
+constexpr int DC_LDP = DC_ROWS + 8;
+constexpr int DC_LDA = DC_ROWS + 4;
+
+struct DeltaChunkArgs {
+    DeltaShape d;
+    DeltaState st;
+    const float* x;           // k_delta_rows<true>: out
+    const float2* gates;
+    const int4* tiles;        // 2 per chunk; the first: (first row, rows, slot, first position)
+    const int4* segs;         // (slot, first position, rows, first row)
+    bf16* w;                  // (M, H, 2, dimp): high and low parts of W
+    float* u;                 // (M, H, vdp)
+    bf16* p;                  // (M, H, 2, 64)
+    float* o;                 // (M, H, vdp)
+    FastDiv row_vecs;         // dimp / 4: 16-byte pieces of a row's high and low parts
+};
+
+// 64 rows of [high | low] parts, n of them valid, into two tiles of padded rows.
+__device__ __forceinline__ void dc_fetch(bf16* dst, const bf16* src, size_t stride, int n, int dimp, const FastDiv& vecs, int n_vecs) {
+    const int ld = dimp + 8, half = n_vecs / 2;
+    for (int i = threadIdx.x; i < DC_ROWS * n_vecs; i += LM_THREADS) {
+        const int r = vecs.div(i), v = i - r * n_vecs;
+        bf16* to = dst + (v < half ? r * ld + v * 8 : (DC_ROWS + r) * ld + (v - half) * 8);
+        cp_async16(to, src + (r < n ? (size_t)r * stride + v * 8 : 0), r < n);
+    }
+}
+
+// d += a b with a and b as (high, low) pairs
+__device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1,
+                                          uint32_t bl0, uint32_t bl1) {
+    mma_bf16(d, ah, bh0, bh1);
+    mma_bf16(d, ah, bl0, bl1);
+    mma_bf16(d, al, bh0, bh1);
+}
+
+static inline size_t delta_solve_smem(int dimp) { return (size_t)4 * DC_ROWS * (dimp + 8) * 2 + (size_t)DC_ROWS * DC_LDA * 4; }
+
+// CTA = (chunk, head).
+static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunkArgs a) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ float G[DC_ROWS], beta[DC_ROWS];
+    pdl_trigger();
+    const DeltaShape& d = a.d;
+    const int ld = d.dimp + 8, nvec = d.dimp / 4;
+    bf16* Ks = reinterpret_cast<bf16*>(smem_raw);              // [2][64][ld]
+    bf16* Qs = Ks + (size_t)2 * DC_ROWS * ld;
+    float* At = reinterpret_cast<float*>(Qs + (size_t)2 * DC_ROWS * ld);   // [s][t], s < t
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.y, kvh = h / (d.H / d.G);
+    pdl_wait();
+    const int4 tile = a.tiles[2 * blockIdx.x];
+    const int row0 = tile.x, n = tile.y;
+    const float* x = a.x + (size_t)row0 * d.C;
+    dc_fetch(Ks, reinterpret_cast<const bf16*>(x + (d.G + kvh) * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
+    dc_fetch(Qs, reinterpret_cast<const bf16*>(x + kvh * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
+    cp_async_commit();
+    if (warp == 0) {
+        float2 gt[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+            gt[i] = 2 * lane + i < n ? __ldcg(a.gates + (size_t)(row0 + 2 * lane + i) * d.H + h) : make_float2(0.f, 0.f);
+        float sum = gt[0].x + gt[1].x;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float v = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += v;
+        }
+        G[2 * lane] = sum - gt[1].x;
+        G[2 * lane + 1] = sum;
+        beta[2 * lane] = gt[0].y;
+        beta[2 * lane + 1] = gt[1].y;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    {   // warps 0-3: keys with keys, 4-7: queries with keys; 16 rows each, columns up to the diagonal
+        const int mt = warp & 3;
+        const bool is_q = warp >= 4;
+        const bf16* A = (is_q ? Qs : Ks) + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
+        const bf16* B = Ks + ((lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
+        float acc[4][2][4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) acc[j][0][i] = acc[j][1][i] = 0.f;
+        for (int ks = 0; ks < d.dimp / 16; ++ks) {
+            uint32_t ah[4], al[4];
+            ldsm_x4(ah, A + ks * 16);
+            ldsm_x4(al, A + DC_ROWS * ld + ks * 16);
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (j <= mt) {
+                    uint32_t bh[4], bl[4];
+                    ldsm_x4(bh, B + j * 16 * ld + ks * 16);
+                    ldsm_x4(bl, B + (DC_ROWS + j * 16) * ld + ks * 16);
+                    mma_split(acc[j][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(acc[j][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                }
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (j <= mt)
+#pragma unroll
+                for (int half = 0; half < 2; ++half)
+#pragma unroll
+                    for (int hi = 0; hi < 2; ++hi) {
+                        const int r = mt * 16 + g + hi * 8, c = j * 16 + half * 8 + 2 * t;
+                        const float v0 = acc[j][half][2 * hi], v1 = acc[j][half][2 * hi + 1], gr = G[r];
+                        if (!is_q) {
+                            if (c < r) At[c * DC_LDA + r] = beta[r] * expf(gr - G[c]) * v0;
+                            if (c + 1 < r) At[(c + 1) * DC_LDA + r] = beta[r] * expf(gr - G[c + 1]) * v1;
+                        } else if (r < n) {
+                            uint32_t ph, pl;
+                            split_bf16x2(c <= r ? expf(gr - G[c]) * v0 : 0.f, c + 1 <= r ? expf(gr - G[c + 1]) * v1 : 0.f, ph, pl);
+                            bf16* p = a.p + ((size_t)(row0 + r) * d.H + h) * 2 * DC_ROWS + c;
+                            *reinterpret_cast<uint32_t*>(p) = ph;
+                            *reinterpret_cast<uint32_t*>(p + DC_ROWS) = pl;
+                        }
+                    }
+    }
+    __syncthreads();
+    // substitution, a thread per column of [beta e^G k | beta v]
+    for (int c = tid; c < d.dimp + d.vdp; c += LM_THREADS) {
+        const bool is_w = c < d.dimp;
+        const int e = is_w ? c : c - d.dimp;
+        float s[DC_ROWS];
+        const float* v = x + 2 * d.G * d.dimp + h * d.vdp + e;
+#pragma unroll
+        for (int i = 0; i < DC_ROWS; ++i)
+            s[i] = is_w ? bf2f(Ks[i * ld + e]) + bf2f(Ks[(DC_ROWS + i) * ld + e]) : i < n ? __ldcg(v + (size_t)i * d.C) : 0.f;
+#pragma unroll
+        for (int i = 0; i < DC_ROWS; ++i) s[i] *= is_w ? beta[i] * expf(G[i]) : beta[i];
+#pragma unroll
+        for (int j = 0; j < DC_ROWS - 1; ++j) {
+            const float xj = -s[j];
+#pragma unroll
+            for (int i = (j + 1) / 4 * 4; i < DC_ROWS; i += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(At + j * DC_LDA + i);
+                if (i > j) s[i] = fmaf(m.x, xj, s[i]);
+                if (i + 1 > j) s[i + 1] = fmaf(m.y, xj, s[i + 1]);
+                if (i + 2 > j) s[i + 2] = fmaf(m.z, xj, s[i + 2]);
+                s[i + 3] = fmaf(m.w, xj, s[i + 3]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < DC_ROWS; ++i)
+            if (i < n) {
+                const size_t row = (size_t)(row0 + i) * d.H + h;
+                if (is_w) {
+                    const bf16 hi = f2bf(s[i]);
+                    a.w[row * 2 * d.dimp + e] = hi;
+                    a.w[row * 2 * d.dimp + d.dimp + e] = f2bf(s[i] - bf2f(hi));
+                } else {
+                    a.u[row * d.vdp + e] = s[i];
+                }
+            }
+    }
+}
+
+template <int NB>
+static inline size_t delta_chunks_smem(int dimp) {
+    return ((size_t)3 * 2 * DC_ROWS * (dimp + 8) + (size_t)2 * DC_ROWS * DC_LDP + (size_t)2 * NB * (dimp + 8) + (size_t)4 * DC_ROWS * (NB + 8)) * 2 +
+           (size_t)DC_ROWS * (NB + 4) * 4;
+}
+
+// CTA = (portion, head, NB value columns).  A warp keeps 16 rows of the state as MMA accumulators.  W, q, U of the next chunk
+// are fetched while this chunk's second half runs, k and P while the next chunk's first half does.
+template <int NB>
+static __global__ void __launch_bounds__(LM_THREADS) k_delta_chunks(DeltaChunkArgs a) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ float eg[DC_ROWS], eg_rest[DC_ROWS];   // e^G_t, e^(G_C - G_t)
+    constexpr int NT = NB / 8, LDV = NB + 8, LDU = NB + 4;
+    pdl_trigger();
+    const DeltaShape& d = a.d;
+    const int ld = d.dimp + 8, nvec = d.dimp / 4, ks_dim = d.dimp / 16;
+    bf16* Ws = reinterpret_cast<bf16*>(smem_raw);      // [2][64][ld], high and low
+    bf16* Qs = Ws + (size_t)2 * DC_ROWS * ld;
+    bf16* Ks = Qs + (size_t)2 * DC_ROWS * ld;
+    bf16* Ps = Ks + (size_t)2 * DC_ROWS * ld;          // [2][64][DC_LDP]
+    bf16* Ss = Ps + (size_t)2 * DC_ROWS * DC_LDP;      // [2][NB][ld], the state by columns
+    bf16* Vs = Ss + (size_t)2 * NB * ld;               // [2][64][LDV]: u
+    bf16* Vd = Vs + (size_t)2 * DC_ROWS * LDV;         // the same times e^(G_C - G_t)
+    float* Us = reinterpret_cast<float*>(Vd + (size_t)2 * DC_ROWS * LDV);   // [64][LDU]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.y, kvh = h / (d.H / d.G), c0 = blockIdx.z * NB, nc = min(NB, d.vdp - c0);   // nc is a multiple of 16
+    pdl_wait();
+    const int4 seg = a.segs[blockIdx.x];
+    const int n_chunks = (seg.z + DC_ROWS - 1) / DC_ROWS;
+    auto fetch_first = [&](int ci) {       // W, q, U
+        if (ci < n_chunks) {
+            const int row0 = seg.w + ci * DC_ROWS, n = min(DC_ROWS, seg.z - ci * DC_ROWS);
+            dc_fetch(Ws, a.w + ((size_t)row0 * d.H + h) * 2 * d.dimp, (size_t)2 * d.H * d.dimp, n, d.dimp, a.row_vecs, nvec);
+            dc_fetch(Qs, reinterpret_cast<const bf16*>(a.x + (size_t)row0 * d.C + kvh * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
+            for (int i = tid; i < DC_ROWS * (NB / 4); i += LM_THREADS) {
+                const int r = i / (NB / 4), v = i % (NB / 4);
+                const bool ok = r < n && 4 * v < nc;
+                cp_async16(Us + r * LDU + v * 4, a.u + (ok ? ((size_t)(row0 + r) * d.H + h) * d.vdp + c0 + v * 4 : 0), ok);
+            }
+        }
+        cp_async_commit();
+    };
+    auto fetch_second = [&](int ci) {      // k, P
+        if (ci < n_chunks) {
+            const int row0 = seg.w + ci * DC_ROWS, n = min(DC_ROWS, seg.z - ci * DC_ROWS);
+            dc_fetch(Ks, reinterpret_cast<const bf16*>(a.x + (size_t)row0 * d.C + (d.G + kvh) * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
+            for (int i = tid; i < DC_ROWS * 16; i += LM_THREADS) {
+                const int r = i >> 4, v = i & 15;
+                cp_async16(Ps + ((v >> 3) * DC_ROWS + r) * DC_LDP + (v & 7) * 8,
+                           a.p + (r < n ? ((size_t)(row0 + r) * d.H + h) * 2 * DC_ROWS + v * 8 : 0), r < n);
+            }
+        }
+        cp_async_commit();
+    };
+    float lg[2];                           // warp 0: log decays of rows 2 * lane, 2 * lane + 1
+    auto ask_gates = [&](int ci) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int r = ci * DC_ROWS + 2 * lane + i;
+            lg[i] = warp == 0 && r < seg.z ? __ldcg(a.gates + (size_t)(seg.w + r) * d.H + h).x : 0.f;
+        }
+    };
+    fetch_first(0);
+    fetch_second(0);
+    ask_gates(0);
+    // the state: rows warp * 16 + g (+ 8), columns c0 + nt * 8 + 2 * t (+ 1)
+    const bool has_s = warp < ks_dim;
+    float* S = a.st.s(seg.x, h, d) + (size_t)c0 * d.dimp + warp * 16 + g;
+    float s[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int col = i * 8 + 2 * t + (e & 1);
+            s[i][e] = has_s && seg.y > 0 && col < nc ? __ldcg(S + (size_t)col * d.dimp + (e >> 1) * 8) : 0.f;
+        }
+    const int mt = warp & 3;
+    const int a_off = (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
+    const int b_off = ((lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
+    const int v_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * LDV + (lane >> 4) * 8;
+    const int kt_off = ((lane & 7) + ((lane >> 4) & 1) * 8) * ld + warp * 16 + ((lane >> 3) & 1) * 8;
+    for (int ci = 0; ci < n_chunks; ++ci) {
+        const int row0 = seg.w + ci * DC_ROWS, n = min(DC_ROWS, seg.z - ci * DC_ROWS);
+        if (has_s)
+#pragma unroll
+            for (int i = 0; i < NT; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    bf16* p = Ss + (i * 8 + 2 * t + (e & 1)) * ld + warp * 16 + g + (e >> 1) * 8;
+                    const bf16 hi = f2bf(s[i][e]);
+                    p[0] = hi;
+                    p[NB * ld] = f2bf(s[i][e] - bf2f(hi));
+                }
+        if (warp == 0) {
+            float sum = lg[0] + lg[1];
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float v = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += v;
+            }
+            const float total = __shfl_sync(0xffffffffu, sum, 31), first = sum - lg[1];
+            eg[2 * lane] = expf(first);
+            eg[2 * lane + 1] = expf(sum);
+            eg_rest[2 * lane] = expf(total - first);
+            eg_rest[2 * lane + 1] = expf(total - sum);
+        }
+        ask_gates(ci + 1);
+        cp_async_wait<1>();
+        __syncthreads();
+        // ---- W S (warps 0-3), q S (warps 4-7)
+        float acc[NT][4];
+#pragma unroll
+        for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+        {
+            const bf16* A = (warp < 4 ? Ws : Qs) + a_off;
+#pragma unroll 2
+            for (int ks = 0; ks < ks_dim; ++ks) {
+                uint32_t ah[4], al[4];
+                ldsm_x4(ah, A + ks * 16);
+                ldsm_x4(al, A + DC_ROWS * ld + ks * 16);
+#pragma unroll
+                for (int j = 0; j < NT / 2; ++j) {
+                    uint32_t bh[4], bl[4];
+                    ldsm_x4(bh, Ss + b_off + j * 16 * ld + ks * 16);
+                    ldsm_x4(bl, Ss + b_off + (NB + j * 16) * ld + ks * 16);
+                    mma_split(acc[2 * j], ah, al, bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(acc[2 * j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+        }
+        const int r_lo = mt * 16 + g, r_hi = r_lo + 8;
+        if (warp < 4) {
+            const float d_lo = eg_rest[r_lo], d_hi = eg_rest[r_hi];
+#pragma unroll
+            for (int i = 0; i < NT; ++i)
+#pragma unroll
+                for (int hi = 0; hi < 2; ++hi) {
+                    const int r = hi ? r_hi : r_lo, c = i * 8 + 2 * t;
+                    const float dd = hi ? d_hi : d_lo;
+                    const float2 u = *reinterpret_cast<const float2*>(Us + r * LDU + c);
+                    const float u0 = u.x - acc[i][2 * hi], u1 = u.y - acc[i][2 * hi + 1];
+                    uint32_t vh, vl;
+                    split_bf16x2(u0, u1, vh, vl);
+                    *reinterpret_cast<uint32_t*>(Vs + r * LDV + c) = vh;
+                    *reinterpret_cast<uint32_t*>(Vs + (DC_ROWS + r) * LDV + c) = vl;
+                    split_bf16x2(u0 * dd, u1 * dd, vh, vl);
+                    *reinterpret_cast<uint32_t*>(Vd + r * LDV + c) = vh;
+                    *reinterpret_cast<uint32_t*>(Vd + (DC_ROWS + r) * LDV + c) = vl;
+                }
+        } else {
+            const float e_lo = eg[r_lo], e_hi = eg[r_hi];
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                acc[i][0] *= e_lo; acc[i][1] *= e_lo;
+                acc[i][2] *= e_hi; acc[i][3] *= e_hi;
+            }
+        }
+        cp_async_wait<0>();      // k and P
+        const float decay = eg[DC_ROWS - 1];
+        __syncthreads();
+        fetch_first(ci + 1);
+        // ---- S = e^G_C S + k^T u
+        if (has_s) {
+#pragma unroll
+            for (int i = 0; i < NT; ++i) { s[i][0] *= decay; s[i][1] *= decay; s[i][2] *= decay; s[i][3] *= decay; }
+#pragma unroll
+            for (int ks = 0; ks < DC_ROWS / 16; ++ks) {
+                uint32_t ah[4], al[4];
+                ldsm_x4_t(ah, Ks + kt_off + ks * 16 * ld);
+                ldsm_x4_t(al, Ks + kt_off + (DC_ROWS + ks * 16) * ld);
+#pragma unroll
+                for (int j = 0; j < NT / 2; ++j) {
+                    uint32_t bh[4], bl[4];
+                    ldsm_x4_t(bh, Vd + v_off + ks * 16 * LDV + j * 16);
+                    ldsm_x4_t(bl, Vd + v_off + (DC_ROWS + ks * 16) * LDV + j * 16);
+                    mma_split(s[2 * j], ah, al, bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(s[2 * j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+        }
+        // ---- o = e^G q S + P u
+        if (warp >= 4) {
+            const bf16* A = Ps + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LDP + (lane >> 4) * 8;
+#pragma unroll
+            for (int ks = 0; ks < DC_ROWS / 16; ++ks)
+                if (ks <= mt) {
+                    uint32_t ah[4], al[4];
+                    ldsm_x4(ah, A + ks * 16);
+                    ldsm_x4(al, A + DC_ROWS * DC_LDP + ks * 16);
+#pragma unroll
+                    for (int j = 0; j < NT / 2; ++j) {
+                        uint32_t bh[4], bl[4];
+                        ldsm_x4_t(bh, Vs + v_off + ks * 16 * LDV + j * 16);
+                        ldsm_x4_t(bl, Vs + v_off + (DC_ROWS + ks * 16) * LDV + j * 16);
+                        mma_split(acc[2 * j], ah, al, bh[0], bh[1], bl[0], bl[1]);
+                        mma_split(acc[2 * j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                    }
+                }
+#pragma unroll
+            for (int i = 0; i < NT; ++i)
+                if (i * 8 < nc) {
+                    float* o = a.o + ((size_t)row0 * d.H + h) * d.vdp + c0 + i * 8 + 2 * t;
+                    if (r_lo < n) *reinterpret_cast<float2*>(o + (size_t)r_lo * d.H * d.vdp) = make_float2(acc[i][0], acc[i][1]);
+                    if (r_hi < n) *reinterpret_cast<float2*>(o + (size_t)r_hi * d.H * d.vdp) = make_float2(acc[i][2], acc[i][3]);
+                }
+        }
+        __syncthreads();         // k, P, u and the state's tiles are used up
+        fetch_second(ci + 1);
+    }
+    if (has_s)
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int col = i * 8 + 2 * t + (e & 1);
+                if (col < nc) S[(size_t)col * d.dimp + (e >> 1) * 8] = s[i][e];
+            }
 }
 
 // ---------------------------------------------------------------------------

@@ -46,6 +46,7 @@ struct LmLayout {
     size_t flag, ctl, row_slot, row_pos, row_ext, segs, xsegs, tiles, x, xn, dq, cq, dkv, gate, q, ay, part, ml, olat;
     size_t tc_partial, tc_counters, xkv, xc;
     size_t raw, dx, dg, dout;   // grouped and delta layers: fp32 rows of the input product; delta: k_delta_rows, recurrence
+    size_t dw, du, dp;          // delta, chunked: k_delta_solve
     size_t draw_ctr, rep_counts, rep_hist, rep_head, rep_filled;
     size_t total;
     int ldx, ld_dq, ld_dkv, ld_gate, ld_ay, ld_q, ld_raw;
@@ -160,6 +161,9 @@ VuibLmDims layer_dims(const VuibLmConfig& c, const VuibLmLayer& l) {
     return d;
 }
 
+// Delta layers whose prefill runs in chunks.
+bool chunked_delta(const VuibLmConfig& c, const VuibLmDims& d) { return c.dtype == VUIB_LM_BF16 && d.dimp <= DC_MAX_DIM; }
+
 int attn_splits(VuibLm* e, int li, int M) {
     const VuibLmLayer& l = e->layer[li];
     const int units = M * ((l.heads + 15) / 16);
@@ -177,7 +181,8 @@ void make_layout(VuibLm* e) {
     const size_t R = e->R, es = c.dtype == VUIB_LM_BF16 ? 2 : 4;
     size_t off = 0;
     auto take = [&](size_t bytes) { size_t o = off; off = align_up(off + bytes); return o; };
-    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0, olat = 0, raw = 0, dx = 0, dg = 0, dout = 0;
+    int dq = 0, cq = 0, dkv = 0, gate = 0, q = 0, ay = 0, xkv = 0, xc = 0, olat = 0, raw = 0, dx = 0, dg = 0, dout = 0, dw = 0;
+    int du = 0, dp = 0;
     size_t part = 0, ml = 0;
     for (size_t i = 0; i < e->layer.size(); ++i) {
         const VuibLmLayer& l = e->layer[i];
@@ -193,6 +198,11 @@ void make_layout(VuibLm* e) {
                 mx(dx, d.n_ab);
                 mx(dg, 2 * l.heads);
                 mx(dout, l.heads * d.vdp);
+                if (chunked_delta(c, d)) {
+                    mx(dw, l.heads * d.dimp);
+                    mx(du, l.heads * d.vdp);
+                    mx(dp, l.heads * DC_ROWS);
+                }
             }
             continue;
         }
@@ -248,6 +258,9 @@ void make_layout(VuibLm* e) {
     L.dx = take(R * dx * 4);
     L.dg = take(R * dg * 4);
     L.dout = take(R * dout * 4);
+    L.dw = take(R * dw * 4);
+    L.du = take(R * du * 4);
+    L.dp = take(R * dp * 4);
     L.draw_ctr = take((size_t)c.n_slots * 4);
     L.rep_counts = take((size_t)c.n_slots * c.vocab * 4);
     L.rep_hist = take((size_t)c.n_slots * REP_HIST_MAX * 4);
@@ -765,13 +778,29 @@ int32_t delta_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
         else RC(run(e, k_delta_step<T, 32, 2>, grid, DT_THREADS, 0, s, ga));
     } else {
         const DeltaRowsArgs ra{ds, dw, st, ga.raw, ga.ldraw, wsp<float>(e, L.dx), wsp<float2>(e, L.dg), row_slot, row_pos, row_ext};
-        RC(run(e, k_delta_rows, dim3(ps.M), LM_THREADS, 0, s, ra));
-        const DeltaScanArgs sa{ds, st, ra.out, ra.gates, wsp<int4>(e, L.segs), wsp<float>(e, L.dout)};
-        const int lpc = d.dimp <= 64 ? 16 : 32, cols = DS_THREADS / lpc * DS_CP;
-        const dim3 grid(ps.n_segs, l.heads, (d.vdp + cols - 1) / cols);
-        if (d.dimp <= 64) RC(run(e, k_delta_scan<16, 1>, grid, DS_THREADS, 0, s, sa));
-        else if (d.dimp <= 128) RC(run(e, k_delta_scan<32, 1>, grid, DS_THREADS, 0, s, sa));
-        else RC(run(e, k_delta_scan<32, 2>, grid, DS_THREADS, 0, s, sa));
+        const bool chunks = ps.n_tiles && chunked_delta(c, d), tile = d.dimp <= 128 && l.taps <= DR_TAPS;
+        const dim3 tiles((ps.M + DR_ROWS - 1) / DR_ROWS);
+        if (tile && chunks) RC(run(e, k_delta_rows_tile<true>, tiles, LM_THREADS, 0, s, ra, ps.M));
+        else if (tile) RC(run(e, k_delta_rows_tile<false>, tiles, LM_THREADS, 0, s, ra, ps.M));
+        else if (chunks) RC(run(e, k_delta_rows<true>, dim3(ps.M), LM_THREADS, 0, s, ra));
+        else RC(run(e, k_delta_rows<false>, dim3(ps.M), LM_THREADS, 0, s, ra));
+        if (chunks) {
+            const DeltaChunkArgs ca{ds, st, ra.out, ra.gates, wsp<int4>(e, L.tiles), wsp<int4>(e, L.segs), wsp<bf16>(e, L.dw), wsp<float>(e, L.du),
+                                    wsp<bf16>(e, L.dp), wsp<float>(e, L.dout), FastDiv(d.dimp / 4)};
+            RC(run(e, k_delta_solve, dim3(ps.n_tiles, l.heads), LM_THREADS, delta_solve_smem(d.dimp), s, ca));
+            const int units = ps.n_segs * l.heads;
+            if (units * ((d.vdp + 31) / 32) >= LS_CTAS)
+                RC(run(e, k_delta_chunks<32>, dim3(ps.n_segs, l.heads, (d.vdp + 31) / 32), LM_THREADS, delta_chunks_smem<32>(d.dimp), s, ca));
+            else
+                RC(run(e, k_delta_chunks<16>, dim3(ps.n_segs, l.heads, d.vdp / 16), LM_THREADS, delta_chunks_smem<16>(d.dimp), s, ca));
+        } else {
+            const DeltaScanArgs sa{ds, st, ra.out, ra.gates, wsp<int4>(e, L.segs), wsp<float>(e, L.dout)};
+            const int lpc = d.dimp <= 64 ? 16 : 32, cols = DS_THREADS / lpc * DS_CP;
+            const dim3 grid(ps.n_segs, l.heads, (d.vdp + cols - 1) / cols);
+            if (d.dimp <= 64) RC(run(e, k_delta_scan<16, 1>, grid, DS_THREADS, 0, s, sa));
+            else if (d.dimp <= 128) RC(run(e, k_delta_scan<32, 1>, grid, DS_THREADS, 0, s, sa));
+            else RC(run(e, k_delta_scan<32, 2>, grid, DS_THREADS, 0, s, sa));
+        }
         RC(run(e, k_delta_gate<T>, dim3(ps.M), LM_THREADS, 0, s, ga));
     }
     return product_out<T>(e, li, ps, s);
