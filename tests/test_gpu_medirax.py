@@ -182,6 +182,24 @@ def test_the_state_remembers_a_far_token(dt, emin):
             assert tm.rel_err(run(eng, ids, cuts)[-1:], want).max() <= min(LIMIT[dtype], 0.2 * seen), (back, cuts)
 
 
+def test_chunks_over_wide_and_narrow_blocks_of_columns():
+    """Enough heads and portions that the chunked recurrence takes its value columns in blocks of 32 and of 64 (one portion,
+    three portions), and few enough that it takes 16; the last block is not full."""
+    for heads in (60, 12):
+        cfg = mm.config([(mm.delta(heads=heads, kv_heads=4, dim=21, vdim=76, conv=3), 40)], width=70)
+        sd = mm.weights(cfg, seed=14)
+        eng = engine(cfg, sd, torch.bfloat16)
+        seqs = [tm.tokens(cfg, n, seed=70 + n) for n in (140, 75, 64, 9)]
+        for group in (seqs[:1], seqs):
+            rows = [eng.new_row() for _ in group]
+            got = eng.step([(r, s, list(range(len(s)))) for r, s in zip(rows, group)])
+            check(got, torch.cat([mm.reference(cfg, sd, s) for s in group]), torch.bfloat16)
+            for x, s, r in zip(eng.step([(r, [5], [0]) for r in rows]), group, rows):
+                check(x[None], mm.reference(cfg, sd, s + [5], [len(s)]), torch.bfloat16)
+                r.close()
+    eng.check_device()
+
+
 @pytest.mark.parametrize("dt", list(DTYPES))
 def test_batches_of_unequal_requests_and_reused_slots(dt):
     """Prefills and decode steps of many rows at once against each row alone (by the oracle), one, few and many rows; then

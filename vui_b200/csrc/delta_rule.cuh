@@ -20,8 +20,8 @@
 // it, unrolling the recurrence gives a unit lower triangular system for the chunk's writes,
 //   (1 + A) u = beta v - (beta e^G k) S_0,   A_ts = beta_t e^(G_t - G_s) k_t . k_s  (s < t),
 //   o_t = e^(G_t) S_0^T q_t + sum_{s <= t} e^(G_t - G_s) (k_s . q_t) u_s,   S_0' = e^(G_C) S_0 + sum_s e^(G_C - G_s) k_s u_s^T.
-// k_delta_solve does what does not need S_0, every chunk on its own: it solves the system for U (right side beta v) and W
-// (right side beta e^G k) by substitution in fp32, and leaves P_ts = e^(G_t - G_s) q_t . k_s.  k_delta_chunks then carries the state
+// k_delta_solve does what does not need S_0, every chunk on its own: it inverts 1 + A in fp32, gives U (right side beta v) and W
+// (right side beta e^G k), and leaves P_ts = e^(G_t - G_s) q_t . k_s.  k_delta_chunks then carries the state
 // from chunk to chunk: u = U - W S_0, o and S_0' as above.  The state stays in fp32 accumulators; a bf16 MMA takes a 32-bit
 // operand as hi + lo bf16 pairs, three products per pair of operands (the product of the two low parts is left out).
 #pragma once
@@ -137,7 +137,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows(DeltaRowsArgs 
     for (int h = threadIdx.x; h < d.H; h += LM_THREADS) a.gates[(size_t)m * d.H + h] = delta_gates(d, a.w, raw, h);
 }
 
-// DR_ROWS consecutive rows per CTA for up to DR_TAPS taps and heads of up to 128: the rows a convolution shares are read once.
+// DR_ROWS consecutive rows and LM_WARPS heads per CTA, for up to DR_TAPS taps and heads of up to 128: the rows a convolution shares are read once.
 constexpr int DR_ROWS = 8, DR_TAPS = 4;
 
 template <bool SPLIT>
@@ -156,7 +156,8 @@ static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows_tile(DeltaRows
     __syncthreads();
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     const int vblocks = (d.H * d.vdp + 127) / 128;
-    for (int i = warp; i < 2 * d.G + vblocks; i += LM_WARPS) {
+    const int i = blockIdx.y * LM_WARPS + warp;
+    if (i < 2 * d.G + vblocks) {
         const bool unit = i < 2 * d.G;      // a query or key head; else 128 value columns
         const int c = unit ? i * d.dimp + 4 * lane : 2 * d.G * d.dimp + (i - 2 * d.G) * 128 + 4 * lane;
         const bool in = unit ? 4 * lane < d.dimp : c < d.C;
@@ -205,7 +206,7 @@ static __global__ void __launch_bounds__(LM_THREADS) k_delta_rows_tile(DeltaRows
             }
         }
     }
-    for (int i = threadIdx.x; i < nr * d.H; i += LM_THREADS) {
+    for (int i = blockIdx.y ? nr * d.H : (int)threadIdx.x; i < nr * d.H; i += LM_THREADS) {
         const int r = i / d.H, h = i - r * d.H;
         a.gates[(size_t)(m0 + r) * d.H + h] = delta_gates(d, a.w, a.raw + (size_t)(m0 + r) * a.ldraw, h);
     }
@@ -353,9 +354,17 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4]
     mma_bf16(d, al, bh0, bh1);
 }
 
-static inline size_t delta_solve_smem(int dimp) { return (size_t)4 * DC_ROWS * (dimp + 8) * 2 + (size_t)DC_ROWS * DC_LDA * 4; }
+constexpr int DC_VCOLS = 128;     // value columns of k_delta_solve in shared memory at a time
+constexpr int DC_LDB = DC_VCOLS + 8;
+constexpr size_t DC_T_BYTES = (size_t)2 * DC_ROWS * DC_LDP * 2;   // a 64 x 64 matrix as (high, low) parts; more than one of floats
+static inline size_t delta_solve_smem(int dimp) {
+    return (size_t)2 * DC_ROWS * (dimp + 8) * 2 + (size_t)2 * DC_ROWS * DC_LDB * 2 + 2 * DC_T_BYTES;
+}
 
-// CTA = (chunk, head).
+// CTA = (chunk, head).  T = (1 + A)^-1 by blocks of 16: the diagonal ones by substitution, a thread per column; the others from
+//   T_ij = -T_ii sum_{j <= k < i} A_ik T_kj
+// one subdiagonal after the other.  Then W = T (beta e^G k) and U = T (beta v) on the tensor cores, the factors of a token moved into
+// T's column.
 static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunkArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ float G[DC_ROWS], beta[DC_ROWS];
@@ -363,8 +372,12 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
     const DeltaShape& d = a.d;
     const int ld = d.dimp + 8, nvec = d.dimp / 4;
     bf16* Ks = reinterpret_cast<bf16*>(smem_raw);              // [2][64][ld]
-    bf16* Qs = Ks + (size_t)2 * DC_ROWS * ld;
-    float* At = reinterpret_cast<float*>(Qs + (size_t)2 * DC_ROWS * ld);   // [s][t], s < t
+    bf16* Bs = Ks + (size_t)2 * DC_ROWS * ld;                  // queries [2][64][ld], then values [2][64][DC_LDB]
+    unsigned char* t0 = reinterpret_cast<unsigned char*>(Bs + (size_t)2 * DC_ROWS * DC_LDB);
+    float* A = reinterpret_cast<float*>(t0);                   // [t][s], s < t
+    float* T = reinterpret_cast<float*>(t0 + DC_T_BYTES);      // [t][s], s <= t by blocks; blocks above hold what is on its way
+    bf16* Tw = reinterpret_cast<bf16*>(t0);                    // T with columns times beta e^G, [2][64][DC_LDP]
+    bf16* Tu = reinterpret_cast<bf16*>(t0 + DC_T_BYTES);       // T with columns times beta
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.y, kvh = h / (d.H / d.G);
     pdl_wait();
@@ -372,7 +385,7 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
     const int row0 = tile.x, n = tile.y;
     const float* x = a.x + (size_t)row0 * d.C;
     dc_fetch(Ks, reinterpret_cast<const bf16*>(x + (d.G + kvh) * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
-    dc_fetch(Qs, reinterpret_cast<const bf16*>(x + kvh * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
+    dc_fetch(Bs, reinterpret_cast<const bf16*>(x + kvh * d.dimp), 2 * d.C, n, d.dimp, a.row_vecs, nvec);
     cp_async_commit();
     if (warp == 0) {
         float2 gt[2];
@@ -395,8 +408,8 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
     {   // warps 0-3: keys with keys, 4-7: queries with keys; 16 rows each, columns up to the diagonal
         const int mt = warp & 3;
         const bool is_q = warp >= 4;
-        const bf16* A = (is_q ? Qs : Ks) + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
-        const bf16* B = Ks + ((lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
+        const bf16* P = (is_q ? Bs : Ks) + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ld + (lane >> 4) * 8;
+        const bf16* K = Ks + ((lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
         float acc[4][2][4];
 #pragma unroll
         for (int j = 0; j < 4; ++j)
@@ -404,14 +417,14 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
             for (int i = 0; i < 4; ++i) acc[j][0][i] = acc[j][1][i] = 0.f;
         for (int ks = 0; ks < d.dimp / 16; ++ks) {
             uint32_t ah[4], al[4];
-            ldsm_x4(ah, A + ks * 16);
-            ldsm_x4(al, A + DC_ROWS * ld + ks * 16);
+            ldsm_x4(ah, P + ks * 16);
+            ldsm_x4(al, P + DC_ROWS * ld + ks * 16);
 #pragma unroll
             for (int j = 0; j < 4; ++j)
                 if (j <= mt) {
                     uint32_t bh[4], bl[4];
-                    ldsm_x4(bh, B + j * 16 * ld + ks * 16);
-                    ldsm_x4(bl, B + (DC_ROWS + j * 16) * ld + ks * 16);
+                    ldsm_x4(bh, K + j * 16 * ld + ks * 16);
+                    ldsm_x4(bl, K + (DC_ROWS + j * 16) * ld + ks * 16);
                     mma_split(acc[j][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
                     mma_split(acc[j][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
                 }
@@ -424,13 +437,13 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
 #pragma unroll
                     for (int hi = 0; hi < 2; ++hi) {
                         const int r = mt * 16 + g + hi * 8, c = j * 16 + half * 8 + 2 * t;
-                        const float v0 = acc[j][half][2 * hi], v1 = acc[j][half][2 * hi + 1], gr = G[r];
+                        const float v0 = c <= r ? expf(G[r] - G[c]) * acc[j][half][2 * hi] : 0.f;
+                        const float v1 = c + 1 <= r ? expf(G[r] - G[c + 1]) * acc[j][half][2 * hi + 1] : 0.f;
                         if (!is_q) {
-                            if (c < r) At[c * DC_LDA + r] = beta[r] * expf(gr - G[c]) * v0;
-                            if (c + 1 < r) At[(c + 1) * DC_LDA + r] = beta[r] * expf(gr - G[c + 1]) * v1;
+                            *reinterpret_cast<float2*>(A + r * DC_LDA + c) = make_float2(c < r ? beta[r] * v0 : 0.f, c + 1 < r ? beta[r] * v1 : 0.f);
                         } else if (r < n) {
                             uint32_t ph, pl;
-                            split_bf16x2(c <= r ? expf(gr - G[c]) * v0 : 0.f, c + 1 <= r ? expf(gr - G[c + 1]) * v1 : 0.f, ph, pl);
+                            split_bf16x2(v0, v1, ph, pl);
                             bf16* p = a.p + ((size_t)(row0 + r) * d.H + h) * 2 * DC_ROWS + c;
                             *reinterpret_cast<uint32_t*>(p) = ph;
                             *reinterpret_cast<uint32_t*>(p + DC_ROWS) = pl;
@@ -438,41 +451,138 @@ static __global__ void __launch_bounds__(LM_THREADS, 2) k_delta_solve(DeltaChunk
                     }
     }
     __syncthreads();
-    // substitution, a thread per column of [beta e^G k | beta v]
-    for (int c = tid; c < d.dimp + d.vdp; c += LM_THREADS) {
-        const bool is_w = c < d.dimp;
-        const int e = is_w ? c : c - d.dimp;
-        float s[DC_ROWS];
-        const float* v = x + 2 * d.G * d.dimp + h * d.vdp + e;
+    // the values of columns v0 .. v0 + 127, by threads first, first + step, ...
+    auto values = [&](int v0, int first, int step) {
+        const float* v = x + 2 * d.G * d.dimp + h * d.vdp + v0;
+        const int cols = min(DC_VCOLS, d.vdp - v0);
+        constexpr int U = 4;
+        for (int i0 = first; i0 < DC_ROWS * (DC_VCOLS / 4); i0 += U * step) {
+            float4 f[U];
 #pragma unroll
-        for (int i = 0; i < DC_ROWS; ++i)
-            s[i] = is_w ? bf2f(Ks[i * ld + e]) + bf2f(Ks[(DC_ROWS + i) * ld + e]) : i < n ? __ldcg(v + (size_t)i * d.C) : 0.f;
-#pragma unroll
-        for (int i = 0; i < DC_ROWS; ++i) s[i] *= is_w ? beta[i] * expf(G[i]) : beta[i];
-#pragma unroll
-        for (int j = 0; j < DC_ROWS - 1; ++j) {
-            const float xj = -s[j];
-#pragma unroll
-            for (int i = (j + 1) / 4 * 4; i < DC_ROWS; i += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(At + j * DC_LDA + i);
-                if (i > j) s[i] = fmaf(m.x, xj, s[i]);
-                if (i + 1 > j) s[i + 1] = fmaf(m.y, xj, s[i + 1]);
-                if (i + 2 > j) s[i + 2] = fmaf(m.z, xj, s[i + 2]);
-                s[i + 3] = fmaf(m.w, xj, s[i + 3]);
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * step, r = i / (DC_VCOLS / 4), c = i % (DC_VCOLS / 4) * 4;
+                f[u] = r < n && c < cols ? __ldcg(reinterpret_cast<const float4*>(v + (size_t)r * d.C + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
-        }
 #pragma unroll
-        for (int i = 0; i < DC_ROWS; ++i)
-            if (i < n) {
-                const size_t row = (size_t)(row0 + i) * d.H + h;
-                if (is_w) {
-                    const bf16 hi = f2bf(s[i]);
-                    a.w[row * 2 * d.dimp + e] = hi;
-                    a.w[row * 2 * d.dimp + d.dimp + e] = f2bf(s[i] - bf2f(hi));
-                } else {
-                    a.u[row * d.vdp + e] = s[i];
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * step, r = i / (DC_VCOLS / 4), c = i % (DC_VCOLS / 4) * 4;
+                if (r < DC_ROWS) {
+                    uint2 hi, lo;
+                    split_bf16x2(f[u].x, f[u].y, hi.x, lo.x);
+                    split_bf16x2(f[u].z, f[u].w, hi.y, lo.y);
+                    *reinterpret_cast<uint2*>(Bs + r * DC_LDB + c) = hi;
+                    *reinterpret_cast<uint2*>(Bs + (DC_ROWS + r) * DC_LDB + c) = lo;
                 }
             }
+        }
+    };
+    if (warp < 2) {
+        const int b = tid & ~15, c = tid & 15;     // block at row b, column c of it
+        float v[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            v[i] = i == c ? 1.f : 0.f;
+#pragma unroll
+            for (int j = 0; j < i; ++j) v[i] = fmaf(-A[(b + i) * DC_LDA + b + j], v[j], v[i]);
+            T[(b + i) * DC_LDA + b + c] = v[i];
+        }
+    } else {
+        values(0, tid - 64, LM_THREADS - 64);
+    }
+    __syncthreads();
+    {
+        const int r = tid >> 4, c = tid & 15;
+        for (int diag = 1; diag < 4; ++diag) {
+            for (int j = 0; j + diag < 4; ++j) {   // sum_k A_ik T_kj, left in the block above the diagonal
+                const int i = j + diag;
+                float v = 0.f;
+                for (int k = 16 * j; k < 16 * i; ++k) v = fmaf(A[(16 * i + r) * DC_LDA + k], T[k * DC_LDA + 16 * j + c], v);
+                T[(16 * j + r) * DC_LDA + 16 * i + c] = v;
+            }
+            __syncthreads();
+            for (int j = 0; j + diag < 4; ++j) {
+                const int i = j + diag;
+                float v = 0.f;
+#pragma unroll
+                for (int k = 0; k < 16; ++k) v = fmaf(T[(16 * i + r) * DC_LDA + 16 * i + k], T[(16 * j + k) * DC_LDA + 16 * i + c], v);
+                T[(16 * i + r) * DC_LDA + 16 * j + c] = -v;
+            }
+            __syncthreads();
+        }
+    }
+    {   // T, scaled, to its (high, low) parts; a thread takes 16 columns of a row
+        const int r = tid >> 2, c0 = (tid & 3) * 16;
+        __align__(16) float v[16];
+#pragma unroll
+        for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(v + i) = *reinterpret_cast<const float4*>(T + r * DC_LDA + c0 + i);
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 16; i += 2) {
+            const int c = c0 + i;
+            const float b0 = v[i] * beta[c], b1 = v[i + 1] * beta[c + 1];
+            uint32_t hi, lo;
+            split_bf16x2(b0, b1, hi, lo);
+            *reinterpret_cast<uint32_t*>(Tu + r * DC_LDP + c) = hi;
+            *reinterpret_cast<uint32_t*>(Tu + (DC_ROWS + r) * DC_LDP + c) = lo;
+            split_bf16x2(b0 * expf(G[c]), b1 * expf(G[c + 1]), hi, lo);
+            *reinterpret_cast<uint32_t*>(Tw + r * DC_LDP + c) = hi;
+            *reinterpret_cast<uint32_t*>(Tw + (DC_ROWS + r) * DC_LDP + c) = lo;
+        }
+        __syncthreads();
+    }
+    // a warp takes 16 columns of W or U at a time
+    const int a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * DC_LDP + (lane >> 4) * 8;
+    auto product = [&](const bf16* M, const bf16* B, int ldb, auto put) {
+        uint32_t bh[4][4], bl[4][4];
+        const bf16* b = B + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldb + (lane >> 4) * 8;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            ldsm_x4_t(bh[ks], b + ks * 16 * ldb);
+            ldsm_x4_t(bl[ks], b + (DC_ROWS + ks * 16) * ldb);
+        }
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt) {
+            float acc[2][4] = {};
+#pragma unroll
+            for (int ks = 0; ks <= mt; ++ks) {
+                uint32_t ah[4], al[4];
+                ldsm_x4(ah, M + a_off + mt * 16 * DC_LDP + ks * 16);
+                ldsm_x4(al, M + a_off + (DC_ROWS + mt * 16) * DC_LDP + ks * 16);
+                mma_split(acc[0], ah, al, bh[ks][0], bh[ks][1], bl[ks][0], bl[ks][1]);
+                mma_split(acc[1], ah, al, bh[ks][2], bh[ks][3], bl[ks][2], bl[ks][3]);
+            }
+#pragma unroll
+            for (int half = 0; half < 2; ++half)
+#pragma unroll
+                for (int hi = 0; hi < 2; ++hi) {
+                    const int r = mt * 16 + g + hi * 8;
+                    if (r < n) put((size_t)(row0 + r) * d.H + h, half * 8 + 2 * t, acc[half][2 * hi], acc[half][2 * hi + 1]);
+                }
+        }
+    };
+    const int w_items = d.dimp / 16;
+    for (int v0 = 0; v0 < d.vdp; v0 += DC_VCOLS) {
+        if (v0) {
+            __syncthreads();
+            values(v0, tid, LM_THREADS);
+            __syncthreads();
+        }
+        const int first = v0 ? w_items : 0, items = w_items + min(DC_VCOLS, d.vdp - v0) / 16;
+        for (int it = first + warp; it < items; it += LM_WARPS) {
+            if (it < w_items) {
+                product(Tw, Ks + it * 16, ld, [&](size_t row, int c, float p0, float p1) {
+                    uint32_t hi, lo;
+                    split_bf16x2(p0, p1, hi, lo);
+                    bf16* w = a.w + row * 2 * d.dimp + it * 16 + c;
+                    *reinterpret_cast<uint32_t*>(w) = hi;
+                    *reinterpret_cast<uint32_t*>(w + d.dimp) = lo;
+                });
+            } else {
+                product(Tu, Bs + (it - w_items) * 16, DC_LDB, [&](size_t row, int c, float p0, float p1) {
+                    *reinterpret_cast<float2*>(a.u + row * d.vdp + v0 + (it - w_items) * 16 + c) = make_float2(p0, p1);
+                });
+            }
+        }
     }
 }
 
@@ -712,37 +822,61 @@ struct DeltaGateArgs {
     const int2* row_ext;
 };
 
-template <class T>
-static __global__ void __launch_bounds__(LM_THREADS) k_delta_gate(DeltaGateArgs<T> a) {
+// A warp takes U (row, head) pairs at a time, P * 128 columns of each.
+template <class T, int P, int U>
+static __global__ void __launch_bounds__(LM_THREADS) k_delta_gate(DeltaGateArgs<T> a, int M) {
     pdl_trigger();
-    pdl_wait();
     const DeltaShape& d = a.d;
-    const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    constexpr int P = DR_MAX_VDIM / 64;
-    for (int h = warp; h < d.H; h += LM_WARPS) {
-        const float* o = a.o + ((size_t)m * d.H + h) * d.vdp;
-        const T* gt = a.gate + (size_t)m * a.ldgate + h * d.vdp;
-        float2 v[P];
-        float ss = 0.f;
+    const int lane = threadIdx.x & 31, i0 = (blockIdx.x * LM_WARPS + (threadIdx.x >> 5)) * U, n = M * d.H;
+    float4 w[P];
+#pragma unroll
+    for (int j = 0; j < P; ++j) w[j] = 4 * lane + 128 * j < d.vdp ? __ldg(reinterpret_cast<const float4*>(a.w.norm) + lane + 32 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    pdl_wait();
+    float4 v[U][P];
+    float gt[U][P][4];
+    int left[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int i = min(i0 + u, n - 1), m = i / d.H, h = i - m * d.H;
+        left[u] = __ldcg(&a.row_ext[m].y);
 #pragma unroll
         for (int j = 0; j < P; ++j) {
-            const int c = 2 * (lane + 32 * j);
-            v[j] = c < d.vdp ? __ldcg(reinterpret_cast<const float2*>(o + c)) : make_float2(0.f, 0.f);
-            ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, ss));
+            const int c = 4 * lane + 128 * j;
+            const bool in = c < d.vdp;
+            v[u][j] = in ? __ldcg(reinterpret_cast<const float4*>(a.o + (size_t)i * d.vdp + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            Store<T>::ld4(a.gate + (size_t)m * a.ldgate + h * d.vdp + (in ? c : 0), gt[u][j]);
         }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        if (i0 + u >= n) break;
+        const int i = i0 + u, m = i / d.H, h = i - m * d.H;
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < P; ++j) ss = dot4(v[u][j], v[u][j], ss);
         const float r = 1.0f / sqrtf(warp_sum(ss) / (float)d.vdim + d.eps);
 #pragma unroll
         for (int j = 0; j < P; ++j) {
-            const int c = 2 * (lane + 32 * j);
+            const int c = 4 * lane + 128 * j;
             if (c < d.vdp)
-                Store<T>::put2(a.out + (size_t)m * a.ldo + h * d.vdp + c, v[j].x * r * __ldg(a.w.norm + c) * Store<T>::ld(gt + c),
-                               v[j].y * r * __ldg(a.w.norm + c + 1) * Store<T>::ld(gt + c + 1));
+                Store<T>::put4(a.out + (size_t)m * a.ldo + h * d.vdp + c,
+                               make_float4(v[u][j].x * r * w[j].x * gt[u][j][0], v[u][j].y * r * w[j].y * gt[u][j][1],
+                                           v[u][j].z * r * w[j].z * gt[u][j][2], v[u][j].w * r * w[j].w * gt[u][j][3]));
         }
-    }
-    if (__ldcg(&a.row_ext[m].y) < d.taps) {
-        const int pos = __ldcg(a.row_pos + m);
-        float* ring = a.st.ring(__ldcg(a.row_slot + m)) + (size_t)(pos % d.taps) * d.C;
-        for (int c = threadIdx.x; c < d.C; c += LM_THREADS) ring[c] = __ldcg(a.raw + (size_t)m * a.ldraw + c);
+        if (left[u] < d.taps) {           // this head's share of the row's channels
+            const int share = (d.C / 4 + d.H - 1) / d.H, end = min(d.C / 4, (h + 1) * share);
+            const float4* raw = reinterpret_cast<const float4*>(a.raw + (size_t)m * a.ldraw);
+            float4* ring = reinterpret_cast<float4*>(a.st.ring(__ldcg(a.row_slot + m)) + (size_t)(__ldcg(a.row_pos + m) % d.taps) * d.C);
+            for (int c0 = h * share + lane; c0 < end; c0 += 4 * 32) {
+                float4 t[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (c0 + 32 * j < end) t[j] = __ldcg(raw + c0 + 32 * j);
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (c0 + 32 * j < end) ring[c0 + 32 * j] = t[j];
+            }
+        }
     }
 }
 

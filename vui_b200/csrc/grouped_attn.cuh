@@ -39,34 +39,39 @@ struct QkHead {        // what a head's components go through after the projecti
     int norm;             // divide by the root mean square
 };
 
-// One warp: a projected head, pairs in adjacent columns, to dst[dimp] (T).
-template <class T>
-__device__ __forceinline__ void qk_head(const QkHead& a, const float* src, int pos, T* dst, int lane, T* dst2 = nullptr) {
-    constexpr int P = GA_MAX_DIM / 64;
-    const float2* tr = a.trig + (size_t)pos * (a.rot_dims / 2);
-    float2 v[P], cs[P];
+// One warp: a projected head, pairs in adjacent columns, in P float2 per lane; rotated and normed in place.
+template <int P>
+__device__ __forceinline__ void qk_load(const QkHead& a, const float* src, int lane, float2 (&v)[P]) {
 #pragma unroll
-    for (int j = 0; j < P; ++j) {
-        const int i = lane + 32 * j;
-        v[j] = 2 * i < a.dimp ? __ldcg(reinterpret_cast<const float2*>(src) + i) : make_float2(0.f, 0.f);
-        cs[j] = 2 * i < a.rot_dims ? __ldg(tr + i) : make_float2(1.f, 0.f);
-    }
+    for (int j = 0; j < P; ++j) v[j] = 2 * (lane + 32 * j) < a.dimp ? __ldcg(reinterpret_cast<const float2*>(src) + lane + 32 * j) : make_float2(0.f, 0.f);
+}
+template <int P>
+__device__ __forceinline__ void qk_turns(const QkHead& a, int pos, int lane, float2 (&cs)[P]) {
+    const float2* tr = a.trig + (size_t)pos * (a.rot_dims / 2);
+#pragma unroll
+    for (int j = 0; j < P; ++j) cs[j] = 2 * (lane + 32 * j) < a.rot_dims ? __ldg(tr + lane + 32 * j) : make_float2(1.f, 0.f);
+}
+template <int P>
+__device__ __forceinline__ void qk_finish(const QkHead& a, const float2 (&cs)[P], float2 (&v)[P]) {
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < P; ++j) {
         v[j] = rotate_pair(v[j].x, v[j].y, cs[j]);
         ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, ss));
     }
-    float r = 1.f;
-    if (a.norm) r = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    if (!a.norm) return;
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
 #pragma unroll
     for (int j = 0; j < P; ++j) {
-        const int i = lane + 32 * j;
-        if (2 * i < a.dimp) {
-            Store<T>::put2(dst + 2 * i, v[j].x * r, v[j].y * r);
-            if (dst2) Store<T>::put2(dst2 + 2 * i, v[j].x * r, v[j].y * r);
-        }
+        v[j].x *= r;
+        v[j].y *= r;
     }
+}
+template <class T, int P>
+__device__ __forceinline__ void qk_put(const QkHead& a, const float2 (&v)[P], T* dst, int lane) {
+#pragma unroll
+    for (int j = 0; j < P; ++j)
+        if (2 * (lane + 32 * j) < a.dimp) Store<T>::put2(dst + 2 * (lane + 32 * j), v[j].x, v[j].y);
 }
 
 struct GroupedCache {
@@ -92,22 +97,65 @@ struct QkRowsArgs {
     int H, G;
 };
 
-template <class T>
-static __global__ void __launch_bounds__(LM_THREADS) k_qk_rows(QkRowsArgs a) {
+// A warp takes U pieces of P * 64 columns of one row: its query heads, its key heads, then pieces of its values.
+static __host__ __device__ __forceinline__ int qk_groups(int H, int G, int vdp, int P, int U) {
+    return (H + G + (G * vdp + 64 * P - 1) / (64 * P) + U - 1) / U;
+}
+
+template <class T, int P, int U>
+static __global__ void __launch_bounds__(LM_THREADS) k_qk_rows(QkRowsArgs a, int M) {
     pdl_trigger();
     pdl_wait();
-    const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int slot = __ldcg(a.row_slot + m), pos = __ldcg(a.row_pos + m), row = ring_row(pos, a.c.cap);
+    const int heads = a.H + a.G, n_v = a.G * a.c.vdp, groups = qk_groups(a.H, a.G, a.c.vdp, P, U);
+    const int lane = threadIdx.x & 31, w = blockIdx.x * LM_WARPS + (threadIdx.x >> 5), m = w / groups, k0 = (w - m * groups) * U;
+    if (m >= M) return;
+    const int pos = __ldcg(a.row_pos + m), slot = __ldcg(a.row_slot + m);
     const float* src = a.raw + (size_t)m * a.ldraw;
-    for (int i = warp; i < a.H + a.G; i += LM_WARPS) {
-        const bool key = i >= a.H;
-        T* dst = key ? a.c.k<T>(slot, i - a.H) + (size_t)row * a.c.dimp : static_cast<T*>(a.q) + ((size_t)m * a.H + i) * a.c.dimp;
-        qk_head<T>(a.h, src + (key ? a.n_k + (i - a.H) * a.c.dimp : i * a.c.dimp), pos, dst, lane);
+    float2 v[U][P], cs[P];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int k = k0 + u;
+        const bool head = k < heads;
+        const float2* p = reinterpret_cast<const float2*>(src + (k < a.H ? k * a.c.dimp : head ? a.n_k + (k - a.H) * a.c.dimp : a.n_v + (k - heads) * 64 * P)) + lane;
+        const int left = head ? a.c.dimp : n_v - (k - heads) * 64 * P;      // columns of this piece
+#pragma unroll
+        for (int j = 0; j < P; ++j) v[u][j] = 2 * (lane + 32 * j) < left ? __ldcg(p + 32 * j) : make_float2(0.f, 0.f);
     }
-    for (int i = 2 * threadIdx.x; i < a.G * a.c.vdp; i += 2 * LM_THREADS) {
-        const int g = i / a.c.vdp, c = i - g * a.c.vdp;
-        const float2 v = __ldcg(reinterpret_cast<const float2*>(src + a.n_v + i));
-        Store<T>::put2(a.c.v<T>(slot, g) + (size_t)row * a.c.vdp + c, v.x, v.y);
+    qk_turns<P>(a.h, pos, lane, cs);
+    float ss[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        ss[u] = 0.f;
+#pragma unroll
+        for (int j = 0; j < P; ++j) {
+            if (k0 + u < heads) v[u][j] = rotate_pair(v[u][j].x, v[u][j].y, cs[j]);
+            ss[u] = fmaf(v[u][j].x, v[u][j].x, fmaf(v[u][j].y, v[u][j].y, ss[u]));
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int u = 0; u < U; ++u) ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o);
+    const int row = ring_row(pos, a.c.cap);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int k = k0 + u;
+        if (k < heads) {
+            const float r = a.h.norm ? 1.0f / sqrtf(ss[u] / (float)a.h.dim + a.h.eps) : 1.f;
+#pragma unroll
+            for (int j = 0; j < P; ++j) {
+                v[u][j].x *= r;
+                v[u][j].y *= r;
+            }
+            qk_put<T, P>(a.h, v[u], k < a.H ? static_cast<T*>(a.q) + ((size_t)m * a.H + k) * a.c.dimp
+                                            : a.c.k<T>(slot, k - a.H) + (size_t)row * a.c.dimp, lane);
+        } else {
+#pragma unroll
+            for (int j = 0; j < P; ++j) {
+                const int c = (k - heads) * 64 * P + 2 * (lane + 32 * j), g = c / a.c.vdp;
+                if (c < n_v) Store<T>::put2(a.c.v<T>(slot, g) + (size_t)row * a.c.vdp + c - g * a.c.vdp, v[u][j].x, v[u][j].y);
+            }
+        }
     }
 }
 
@@ -216,15 +264,20 @@ static __global__ void __launch_bounds__(LM_THREADS) k_grouped_attn(GroupedAttnA
             const float* src = a.r.raw + (size_t)m * a.r.ldraw;
             const int row = ring_row(pos, cap);
             const bool store = owner && hg == 0;
+            constexpr int P = GA_MAX_DIM / 64;
+            float2 cs[P], v[P];
+            qk_turns<P>(a.r.h, pos, lane, cs);
             for (int i = warp; i < 17; i += LM_WARPS) {
-                if (i < nh) {
-                    qk_head<bf16>(a.r.h, src + (h0 + i) * dimp, pos, Qs + i * ldk, lane);
-                } else if (i < 16) {
-                    for (int c = lane; c < dimp / 2; c += 32) reinterpret_cast<uint32_t*>(Qs + i * ldk)[c] = 0u;
-                } else if (owner) {
-                    qk_head<bf16>(a.r.h, src + a.r.n_k + kvh * dimp, pos, own_k, lane,
-                                  store ? a.r.c.k<bf16>(slot, kvh) + (size_t)row * dimp : nullptr);
+                const int q = i == LM_WARPS - 1 ? 16 : i == 16 ? LM_WARPS - 1 : i;     // the key is the last warp's first
+                if (q >= nh && q < 16) {
+                    for (int c = lane; c < dimp / 2; c += 32) reinterpret_cast<uint32_t*>(Qs + q * ldk)[c] = 0u;
+                    continue;
                 }
+                if (q == 16 && !owner) continue;
+                qk_load<P>(a.r.h, src + (q < 16 ? (h0 + q) * dimp : a.r.n_k + kvh * dimp), lane, v);
+                qk_finish<P>(a.r.h, cs, v);
+                qk_put<bf16, P>(a.r.h, v, q < 16 ? Qs + q * ldk : own_k, lane);
+                if (q == 16 && store) qk_put<bf16, P>(a.r.h, v, a.r.c.k<bf16>(slot, kvh) + (size_t)row * dimp, lane);
             }
             if (owner)
                 for (int c = 2 * tid; c < vdp; c += 2 * LM_THREADS) {

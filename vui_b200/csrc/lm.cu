@@ -712,6 +712,15 @@ int32_t grouped_tiles(VuibLm* e, const GroupedPrefillArgs& a, int n_tiles, cudaS
 }
 
 template <class T>
+int32_t qk_rows(VuibLm* e, const QkRowsArgs& r, int M, cudaStream_t s) {
+    const int p = r.c.dimp <= 64 ? 1 : r.c.dimp <= 128 ? 2 : 4, u = 8 / p;
+    const dim3 grid((M * qk_groups(r.H, r.G, r.c.vdp, p, u) + LM_WARPS - 1) / LM_WARPS);
+    if (p == 1) return run(e, k_qk_rows<T, 1, 8>, grid, LM_THREADS, 0, s, r, M);
+    if (p == 2) return run(e, k_qk_rows<T, 2, 4>, grid, LM_THREADS, 0, s, r, M);
+    return run(e, k_qk_rows<T, 4, 2>, grid, LM_THREADS, 0, s, r, M);
+}
+
+template <class T>
 int32_t grouped_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
     const VuibLmConfig& c = e->cfg;
     const LmLayout& L = e->lay;
@@ -736,7 +745,7 @@ int32_t grouped_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
         if (ps.step) {
             RC(grouped_rows_bf16<true>(e, li, r, ps.M, s));
         } else {
-            RC(run(e, k_qk_rows<T>, dim3(ps.M), LM_THREADS, 0, s, r));
+            RC(qk_rows<T>(e, r, ps.M, s));
             if (ps.n_tiles) {
                 const GroupedPrefillArgs a{static_cast<const bf16*>(r.q), r.c, wsp<int4>(e, L.tiles), wsp<bf16>(e, L.ay), L.ld_ay, l.heads,
                                            hpg, window, l.scale, l.softcap, FastDiv((d.dimp + d.vdp) / 8)};
@@ -748,7 +757,7 @@ int32_t grouped_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
             }
         }
     } else {
-        RC(run(e, k_qk_rows<T>, dim3(ps.M), LM_THREADS, 0, s, r));
+        RC(qk_rows<T>(e, r, ps.M, s));
         const GroupedAttnF32Args a{static_cast<const float*>(r.q), r.c, r.row_slot, r.row_pos, wsp<float>(e, L.ay), L.ld_ay, l.heads, hpg,
                                    window, l.scale, l.softcap};
         RC(run(e, k_grouped_attn_f32, dim3(ps.M, l.heads), LM_THREADS, 0, s, a));
@@ -779,7 +788,7 @@ int32_t delta_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
     } else {
         const DeltaRowsArgs ra{ds, dw, st, ga.raw, ga.ldraw, wsp<float>(e, L.dx), wsp<float2>(e, L.dg), row_slot, row_pos, row_ext};
         const bool chunks = ps.n_tiles && chunked_delta(c, d), tile = d.dimp <= 128 && l.taps <= DR_TAPS;
-        const dim3 tiles((ps.M + DR_ROWS - 1) / DR_ROWS);
+        const dim3 tiles((ps.M + DR_ROWS - 1) / DR_ROWS, (2 * l.kv_heads + (l.heads * d.vdp + 127) / 128 + LM_WARPS - 1) / LM_WARPS);
         if (tile && chunks) RC(run(e, k_delta_rows_tile<true>, tiles, LM_THREADS, 0, s, ra, ps.M));
         else if (tile) RC(run(e, k_delta_rows_tile<false>, tiles, LM_THREADS, 0, s, ra, ps.M));
         else if (chunks) RC(run(e, k_delta_rows<true>, dim3(ps.M), LM_THREADS, 0, s, ra));
@@ -789,7 +798,9 @@ int32_t delta_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
                                     wsp<bf16>(e, L.dp), wsp<float>(e, L.dout), FastDiv(d.dimp / 4)};
             RC(run(e, k_delta_solve, dim3(ps.n_tiles, l.heads), LM_THREADS, delta_solve_smem(d.dimp), s, ca));
             const int units = ps.n_segs * l.heads;
-            if (units * ((d.vdp + 31) / 32) >= LS_CTAS)
+            if (units * ((d.vdp + 63) / 64) >= LS_CTAS)
+                RC(run(e, k_delta_chunks<64>, dim3(ps.n_segs, l.heads, (d.vdp + 63) / 64), LM_THREADS, delta_chunks_smem<64>(d.dimp), s, ca));
+            else if (units * ((d.vdp + 31) / 32) >= LS_CTAS)
                 RC(run(e, k_delta_chunks<32>, dim3(ps.n_segs, l.heads, (d.vdp + 31) / 32), LM_THREADS, delta_chunks_smem<32>(d.dimp), s, ca));
             else
                 RC(run(e, k_delta_chunks<16>, dim3(ps.n_segs, l.heads, d.vdp / 16), LM_THREADS, delta_chunks_smem<16>(d.dimp), s, ca));
@@ -801,7 +812,9 @@ int32_t delta_layer(VuibLm* e, int li, const Pass& ps, cudaStream_t s) {
             else if (d.dimp <= 128) RC(run(e, k_delta_scan<32, 1>, grid, DS_THREADS, 0, s, sa));
             else RC(run(e, k_delta_scan<32, 2>, grid, DS_THREADS, 0, s, sa));
         }
-        RC(run(e, k_delta_gate<T>, dim3(ps.M), LM_THREADS, 0, s, ga));
+        const int items = ps.M * l.heads;
+        if (d.vdp <= 128) RC(run(e, k_delta_gate<T, 1, 4>, dim3((items + 4 * LM_WARPS - 1) / (4 * LM_WARPS)), LM_THREADS, 0, s, ga, ps.M));
+        else RC(run(e, k_delta_gate<T, 4, 1>, dim3((items + LM_WARPS - 1) / LM_WARPS), LM_THREADS, 0, s, ga, ps.M));
     }
     return product_out<T>(e, li, ps, s);
 }

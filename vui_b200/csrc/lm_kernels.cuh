@@ -28,12 +28,26 @@ template <> struct Store<bf16> {
         *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
     }
     static __device__ __forceinline__ void unpack(const uint4& u, float (&f)[8]) { unpack8(u, f); }
+    static __device__ __forceinline__ void ld4(const bf16* p, float (&f)[4]) {
+        const uint2 u = __ldcg(reinterpret_cast<const uint2*>(p));
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+    }
+    static __device__ __forceinline__ void put4(bf16* p, const float4& v) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
 };
 template <> struct Store<float> {
     static constexpr int VEC = 4;
     static __device__ __forceinline__ float ld(const float* p) { return *p; }
     static __device__ __forceinline__ void put(float* p, float v) { *p = v; }
     static __device__ __forceinline__ void put2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+    static __device__ __forceinline__ void ld4(const float* p, float (&f)[4]) {
+        const float4 v = __ldcg(reinterpret_cast<const float4*>(p));
+        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+    }
+    static __device__ __forceinline__ void put4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
     static __device__ __forceinline__ void unpack(const uint4& u, float (&f)[4]) {
         f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y);
         f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
